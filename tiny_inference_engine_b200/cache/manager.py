@@ -13,7 +13,9 @@ per group: token j lives in page table[j // page_size] at offset j % page_size
 
 Pages go back to the pool when a request is released (finished, cancelled or preempted),
 when a table is truncated after a failed step, and, in a window group, when the window has
-passed them: their table entry becomes -1 and no later query reads below the window.
+passed them: their table entry becomes -1 and no later query reads below the window. A window group
+may keep a sequence's first tokens beside the window (`keep_first`): the pages that hold them stay
+until the request ends.
 `reserve` is all-or-nothing over all groups (src/kv/paged_kv_cache.cpp:41-49).
 
 A request that only waits holds nothing (src/engine/sequence.h:15-30: an empty block table):
@@ -44,12 +46,13 @@ def blocks_for(tokens: int, page_size: int) -> int:
 
 class BlockTable:
     """Page ids of one request in one group, in a numpy array so that a step can copy it fast."""
-    __slots__ = ("ids", "n", "released")
+    __slots__ = ("ids", "n", "released", "kept")
 
-    def __init__(self):
+    def __init__(self, kept: int = 0):
         self.ids = np.empty(16, dtype=np.int32)
         self.n = 0          # entries in use (positional: entry i covers tokens [i*page, (i+1)*page))
-        self.released = 0   # leading entries already given back (window groups)
+        self.released = 0   # leading entries the window has passed (window groups): given back, but for the kept ones
+        self.kept = kept    # leading entries that are never given back while the request lives
 
     def append(self, block: int) -> None:
         if self.n == len(self.ids):
@@ -61,7 +64,11 @@ class BlockTable:
         return self.ids[:self.n]
 
     def held(self) -> list[int]:
-        return [int(b) for b in self.ids[self.released:self.n]]
+        kept = min(self.kept, self.released, self.n)
+        return [int(b) for b in self.ids[:kept]] + [int(b) for b in self.ids[self.released:self.n]]
+
+    def holds(self) -> bool:
+        return self.n > self.released or min(self.kept, self.n) > 0
 
     def __len__(self) -> int:
         return self.n
@@ -83,6 +90,7 @@ class GroupSpec:
     window: int
     entries: tuple[int, ...]   # run entries whose planes live in this group
     value_dim: int = 0         # size of a value head; 0: head_dim; VALUES_IN_KEYS: no value plane
+    keep_first: int = 0        # "window": the sequence's first tokens that stay beside the window
 
 
 class CacheManager:
@@ -105,11 +113,13 @@ class CacheManager:
                 continue
             value_dim = getattr(need, "value_dim", 0)
             if need.kv_heads <= 0 or need.head_dim <= 0 or value_dim < VALUES_IN_KEYS or need.kind not in ("full", "window") or \
-                    (need.kind == "window" and need.window <= 0):
+                    (need.kind == "window" and need.window <= 0) or getattr(need, "keep_first", 0) < 0:
                 raise InvalidArgument(f"bad cache need of run entry {i}: {need}")
             keyed.setdefault((need.kind, need.kv_heads, need.head_dim, need.window if need.kind == "window" else 0,
-                              0 if value_dim == need.head_dim else value_dim), []).append(i)
-        self.groups = [GroupSpec(k[0], k[1], k[2], k[3], tuple(v), k[4]) for k, v in keyed.items()]
+                              0 if value_dim == need.head_dim else value_dim,
+                              getattr(need, "keep_first", 0) if need.kind == "window" else 0), []).append(i)
+        self.groups = [GroupSpec(k[0], k[1], k[2], k[3], tuple(v), k[4], k[5]) for k, v in keyed.items()]
+        self._kept_pages = [blocks_for(g.keep_first, page_size) for g in self.groups]
         self._entry_group = {e: gi for gi, g in enumerate(self.groups) for e in g.entries}
         self._entry_plane = {e: pi for g in self.groups for pi, e in enumerate(g.entries)}
         elem = 4 if dtype is None else _elem_size(dtype)
@@ -121,7 +131,7 @@ class CacheManager:
                 raise InvalidArgument(f"bad window sizing: {window_requests} requests, {window_step_tokens} tokens a step")
             for gi, g in enumerate(self.groups):
                 if g.kind == "window":
-                    bounded[gi] = window_requests * (blocks_for(g.window + window_step_tokens, page_size) + 2)
+                    bounded[gi] = window_requests * (blocks_for(g.window + window_step_tokens, page_size) + 2 + self._kept_pages[gi])
         self.bytes_per_page = sum(b for b, fixed in zip(group_bytes, bounded) if fixed is None) or sum(group_bytes)
         if num_pages is None:
             if budget_bytes is None:
@@ -163,7 +173,7 @@ class CacheManager:
     # -- requests
     def new_request(self) -> RequestCache:
         """A request that holds nothing yet: empty tables, no state slot."""
-        req = RequestCache([BlockTable() for _ in self.groups], -1)
+        req = RequestCache([BlockTable(kept) for kept in self._kept_pages], -1)
         self._live.add(id(req))
         return req
 
@@ -182,7 +192,7 @@ class CacheManager:
 
     def holds(self, req: RequestCache) -> bool:
         """Whether preempting the request would give anything back: a page or a state slot."""
-        return req.state_slot >= 0 or any(len(t) > t.released for t in req.tables)
+        return req.state_slot >= 0 or any(t.holds() for t in req.tables)
 
     def room(self, req: RequestCache, computed: int) -> int:
         """How many more tokens `req` could hold with its pages plus all free ones
@@ -247,15 +257,16 @@ class CacheManager:
     def advance_window(self, req: RequestCache, computed: int) -> None:
         """After `computed` tokens are in the cache, window groups give back every page that no
         later query can read: the next query is at position >= computed and reads keys
-        > position - window."""
+        > position - window (and the first `keep_first`, whose pages stay)."""
         for g, t, p in zip(self.groups, req.tables, self.pools):
             if g.kind != "window":
                 continue
             first_needed = max(0, computed - g.window + 1)
             upto = min(first_needed // self.page_size, t.n)
             while t.released < upto:
-                p.release(int(t.ids[t.released]))
-                t.ids[t.released] = FREED
+                if t.released >= t.kept:
+                    p.release(int(t.ids[t.released]))
+                    t.ids[t.released] = FREED
                 t.released += 1
 
     def release(self, req: RequestCache) -> None:

@@ -58,6 +58,9 @@ struct DecodeArgs {
   float q_eps, k_eps;
   const int* positions;
   __nv_bfloat16 *k_plane, *v_plane;
+  int keep_first;        // the sequence's first keys that stay visible beside a window: split 0 reads them
+  float softcap;         // > 0: score <- softcap * tanh(score / softcap)
+  const float* sink;     // [q_heads] or null: exp(sink[h]) is one more term of the softmax's denominator, without a value
 };
 
 // A float into the shared memory of another CTA of the cluster (`mine`: the address in this CTA's own).
@@ -141,7 +144,12 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
     return;
   }
   const int kt_first = lo / kKeysPerTile, kt_last = hi / kKeysPerTile;
-  const int n_tiles = no_keys ? 0 : kt_last - kt_first + 1;
+  // Kept keys below the window belong to split 0: the tiles that hold them come ahead of the split's own (a tile that the
+  // split reads anyway is not read twice).
+  const int kept = split == 0 ? min(a.keep_first, lo0) : 0;
+  const int kept_tiles = min((kept + kKeysPerTile - 1) / kKeysPerTile, kt_first);
+  const int n_tiles = no_keys ? 0 : kt_last - kt_first + 1 + kept_tiles;
+  const auto tile_of = [&](int i) { return i < kept_tiles ? i : kt_first + i - kept_tiles; };
   const int box_rows = min(a.page_size, kKeysPerTile);
   const int boxes_per_tile = kKeysPerTile / box_rows;
 
@@ -159,9 +167,8 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
   // and keys beyond `hi` are masked, so what it holds does not matter as long as it is finite
   if (a.window > 0) {
     const int* table = a.block_tables + static_cast<long long>(seq) * a.max_blocks;
-    const int first_key = kt_first * kKeysPerTile;
     for (int b = threadIdx.x; b < n_tiles * boxes_per_tile; b += kDecThreads) {
-      const int idx = (first_key + b * box_rows) >> a.page_shift;
+      const int idx = (tile_of(b / boxes_per_tile) * kKeysPerTile + b % boxes_per_tile * box_rows) >> a.page_shift;
       pages[b] = idx < a.max_blocks ? table[idx] : 0;
     }
   } else {
@@ -194,7 +201,7 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
       uint8_t* kdst = smem + s * STAGE_BYTES;
       for (int op = lane; op < ops_per_tile; op += 32) {
         const int b = op / (2 * HALVES), h = (op % (2 * HALVES)) >> 1, is_v = op & 1;
-        const int key = (kt_first + i) * kKeysPerTile + b * box_rows;
+        const int key = tile_of(i) * kKeysPerTile + b * box_rows;
         const int row = (pages[i * boxes_per_tile + b] * a.kv_heads + kvh) * a.page_size + (key & (a.page_size - 1));
         tma_load_2d(kdst + is_v * PLANE_BYTES + h * (64 * 128) + b * box_rows * 128, is_v ? &v_map : &k_map, h * 64, row, full + s);
       }
@@ -246,7 +253,7 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
           *reinterpret_cast<Slice*>(q_tile + RowLayout<DH>::at(r, (lane * VEC) >> 3) + ((lane * VEC * 2) & 15)) = out;
         } else {
           // the page of the newest key is among this split's pages; the same row the TMA boxes of that page start from
-          const int box = (pos - kt_first * kKeysPerTile) / box_rows;
+          const int box = (pos - kt_first * kKeysPerTile) / box_rows + kept_tiles * boxes_per_tile;
           const long long row = static_cast<long long>(pages[box] * a.kv_heads + kvh) * a.page_size + (pos & (a.page_size - 1));
           *reinterpret_cast<Slice*>((r == G ? a.k_plane : a.v_plane) + row * DH + lane * VEC) = out;
           *reinterpret_cast<Slice*>(newest + (r - G) * DH + lane * VEC) = out;
@@ -273,7 +280,7 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
       if constexpr (PREP) {
         // The tile came from the cache as it was before this step: the newest key's row gets what this kernel made,
         // from the warp that works on that key (no other warp reads the row).
-        const int rr = pos - (kt_first + i) * kKeysPerTile;
+        const int rr = pos - tile_of(i) * kKeysPerTile;
         if (appends && i == n_tiles - 1 && warp == (rr >> 4)) {
           uint8_t* tile = smem + s * STAGE_BYTES;
           const uint32_t at = L::at(rr, (lane * VEC) >> 3) + ((lane * VEC * 2) & 15);
@@ -282,8 +289,8 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
           __syncwarp();
         }
       }
-      const int key0 = (kt_first + i) * kKeysPerTile + warp * 16;   // this warp's 16 keys of the tile
-      if (key0 <= hi && key0 + 15 >= lo) {
+      const int key0 = tile_of(i) * kKeysPerTile + warp * 16;   // this warp's 16 keys of the tile
+      if (key0 <= hi && (key0 + 15 >= lo || key0 < kept)) {
         const uint32_t k_tile = smem_u32(smem + s * STAGE_BYTES);
         float sc[2][4];
 #pragma unroll
@@ -294,7 +301,11 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int key = key0 + j * 8 + tq * 2 + (e & 1);
-            sc[j][e] = (key >= lo && key <= hi) ? sc[j][e] * a.scale_log2 : -INFINITY;
+            float v = sc[j][e] * a.scale_log2;
+            // (float arithmetic on the fast exponential, as in the prompt kernel: tanh(z) = 1 - 2 / (exp(2 z) + 1))
+            if (a.softcap > 0.0f)
+              v = a.softcap * 1.4426950408889634f * (1.0f - __fdividef(2.0f, exp2f(2.0f * v / a.softcap) + 1.0f));
+            sc[j][e] = ((key >= lo && key <= hi) || key < kept) ? v : -INFINITY;
           }
         }
         softmax_update<DH, 2>(sc, m, l, acc);
@@ -349,6 +360,13 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
       fac[r * 4 + w] = f;
       ls += part[(w * 16 + r) * RS + DH + 1] * f;
     }
+    if (a.sink != nullptr && n_splits == 1) {      // with several splits the merge adds it, once
+      const float sink = a.sink[kvh * G + r] * 1.4426950408889634f, top = fmaxf(mx, sink), f = exp2f(mx - top);
+      ls = fmaf(ls, f, exp2f(sink - top));
+#pragma unroll
+      for (int w = 0; w < 4; ++w) fac[r * 4 + w] *= f;
+      mx = top;
+    }
     fac[4 * G + r] = mx;
     fac[5 * G + r] = ls;
   }
@@ -380,6 +398,11 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
           float mx = -INFINITY;
           for (int i = 0; i < n_splits; ++i) mx = fmaxf(mx, mine[i * RS + DH]);
           float ls = 0.0f;
+          if (a.sink != nullptr) {
+            const float sink = a.sink[kvh * G + r] * 1.4426950408889634f;
+            mx = fmaxf(mx, sink);
+            ls = exp2f(sink - mx);
+          }
           for (int i = 0; i < n_splits; ++i) {
             const float w = exp2f(mine[i * RS + DH] - mx);
             wgt[i] = w;
@@ -448,6 +471,11 @@ __global__ void __launch_bounds__(kDecThreads) attn_decode_tma_kernel(const __gr
     float mx = -INFINITY;
     for (int i = 0; i < n_splits; ++i) mx = fmaxf(mx, msm[r * a.max_splits + i]);
     float ls = 0.0f;
+    if (a.sink != nullptr) {
+      const float sink = a.sink[kvh * G + r] * 1.4426950408889634f;
+      mx = fmaxf(mx, sink);
+      ls = exp2f(sink - mx);
+    }
     for (int i = 0; i < n_splits; ++i) {
       const float w = exp2f(msm[r * a.max_splits + i] - mx);
       wgt[r * a.max_splits + i] = w;
@@ -549,7 +577,9 @@ static int decode_tma(DecodeArgs a, bool prep, bool cluster, const void* k_cache
   TIE_REQUIRE(split_keys > 0 && split_keys % kKeysPerTile == 0 && max_splits > 0 && a.scratch != nullptr && a.counters != nullptr,
               "attention_decode: splits must be positive multiples of %d keys", kKeysPerTile);
   const int box_rows = page_size < kKeysPerTile ? page_size : kKeysPerTile;
-  TIE_REQUIRE((split_keys / kKeysPerTile + 1) * (kKeysPerTile / box_rows) <= kMaxTablePages && max_splits <= 256,
+  TIE_REQUIRE(a.keep_first == 0 || a.window > 0, "attention_decode: kept keys go with a window");
+  const int kept_tiles = (a.keep_first + kKeysPerTile - 1) / kKeysPerTile;
+  TIE_REQUIRE((split_keys / kKeysPerTile + 1 + kept_tiles) * (kKeysPerTile / box_rows) <= kMaxTablePages && max_splits <= 256,
               "attention_decode: a split of %d keys over pages of %d (or %d splits) exceeds the kernel's tables", split_keys,
               page_size, max_splits);
   if (n_list == 0) return kOk;
@@ -596,7 +626,8 @@ static int decode_tma_plain(const void* q, long long q_stride, const void* k_cac
                             const int* query_start, const int* context_lens, const int* block_tables, int max_blocks,
                             int q_heads, int kv_heads, int head_dim, int page_size, int pages, int window, float scale,
                             const int* seq_list, int seq_first, int n_list, int split_keys, int max_splits, float* scratch,
-                            int* counters, int cluster, int exact_weights, cudaStream_t s) {
+                            int* counters, int cluster, int exact_weights, cudaStream_t s, int keep_first = 0, float softcap = 0.0f,
+                            const float* sink = nullptr) {
   TIE_REQUIRE(q_stride % 8 == 0 && reinterpret_cast<uintptr_t>(q) % 16 == 0, "attention_decode: q rows must be 16-byte aligned");
   DecodeArgs a{};
   a.q = static_cast<const __nv_bfloat16*>(q);
@@ -605,6 +636,7 @@ static int decode_tma_plain(const void* q, long long q_stride, const void* k_cac
   a.scratch = scratch, a.counters = counters, a.q_stride = q_stride;
   a.max_blocks = max_blocks, a.q_heads = q_heads, a.kv_heads = kv_heads, a.page_size = page_size, a.window = window;
   a.split_keys = split_keys, a.max_splits = max_splits, a.exact_weights = exact_weights;
+  a.keep_first = keep_first, a.softcap = softcap, a.sink = sink;
   return decode_tma(a, false, cluster != 0, k_cache, v_cache, head_dim, pages, n_list, scale, s);
 }
 
@@ -629,6 +661,19 @@ TIE_API int tie_attention_decode_tma_exact(const void* q, long long q_stride, co
   return decode_tma_plain(q, q_stride, k_cache, v_cache, out, query_start, context_lens, block_tables, max_blocks, q_heads, kv_heads,
                           head_dim, page_size, pages, window, scale, seq_list, seq_first, n_list, split_keys, max_splits, scratch,
                           counters, cluster, 1, s);
+}
+
+// A window beside which the sequence's first keys stay visible, capped scores (softcap, 0: none) and a sink per head (null:
+// none), with the softmax weights kept to 16 bits of mantissa.
+TIE_API int tie_attention_decode_kept(const void* q, long long q_stride, const void* k_cache, const void* v_cache, void* out,
+                                      const int* query_start, const int* context_lens, const int* block_tables, int max_blocks,
+                                      int q_heads, int kv_heads, int head_dim, int page_size, int pages, int window, int keep_first,
+                                      float scale, float softcap, const float* sink, const int* seq_list, int seq_first, int n_list,
+                                      int split_keys, int max_splits, float* scratch, int* counters, int cluster, cudaStream_t s) {
+  TIE_REQUIRE(keep_first >= 0 && softcap >= 0.0f, "attention_decode: %d kept keys, a cap of %g", keep_first, static_cast<double>(softcap));
+  return decode_tma_plain(q, q_stride, k_cache, v_cache, out, query_start, context_lens, block_tables, max_blocks, q_heads, kv_heads,
+                          head_dim, page_size, pages, window, scale, seq_list, seq_first, n_list, split_keys, max_splits, scratch,
+                          counters, cluster, 1, s, keep_first, softcap, sink);
 }
 
 // The same attention for a step in which every sequence brings one token, straight from the output of the q/k/v

@@ -42,6 +42,8 @@ struct PromptArgs {
   const float* r1;        // [q_heads] or null: score -= r1[h] * ln(1 + r2[h] * (position - key position))
   const float* r2;
   int out_f32;            // != 0: `out` holds float rows (what follows combines heads' outputs and wants them unrounded)
+  int keep_first;         // the sequence's first keys that stay visible beside a window
+  const float* sink;      // [q_heads] or null: exp(sink[h]) is one more term of the softmax's denominator, without a value
 };
 
 // The first key that position `pos` sees.
@@ -85,7 +87,11 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
   const int v_slices = a.v_ld > 0 ? a.v_ld / DH : 1;
   const int v_slice = (kvh / cache_heads + a.v_shift) % v_slices, v_col = v_slice * DH;
   const int kt_first = lo_cta / kKeysPerTile, kt_last = hi_cta / kKeysPerTile;
-  const int n_tiles = kt_last - kt_first + 1;
+  // Ahead of the window's tiles: the tiles that hold kept keys some row of the CTA does not see through its window.
+  const int kept = min(a.keep_first, prompt_first_visible(hi_cta, a.window, a.chunk));
+  const int kept_tiles = min((kept + kKeysPerTile - 1) / kKeysPerTile, kt_first);
+  const int n_tiles = kt_last - kt_first + 1 + kept_tiles;
+  const auto tile_of = [&](int i) { return i < kept_tiles ? i : kt_first + i - kept_tiles; };
   const int box_rows = min(a.page_size, kKeysPerTile);
   const int boxes_per_tile = kKeysPerTile / box_rows;
   const int* table = a.block_tables + static_cast<long long>(seq) * a.max_blocks;
@@ -132,7 +138,7 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
       ok = __shfl_sync(0xffffffffu, ok, 0);
       if (!ok) break;
       if (lane < boxes_per_tile) {
-        const int key = (kt_first + i) * kKeysPerTile + lane * box_rows;
+        const int key = tile_of(i) * kKeysPerTile + lane * box_rows;
         const int idx = key >> a.page_shift;
         const int page = idx < a.max_blocks ? table[idx] : 0;   // beyond the table: any real page; those keys are masked
         const int row = (page * cache_heads + cached_head) * a.page_size + (key & (a.page_size - 1));
@@ -169,8 +175,8 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
     for (int i = 0; i < n_tiles; ++i) {
       const int s = i % STAGES;
       if (!mbar_wait(full + s, (i / STAGES) & 1, abort_flag, a.status, 12)) break;
-      const int key0 = (kt_first + i) * kKeysPerTile;
-      const bool in_window = !limited || key0 + 63 >= prompt_first_visible(warp_lo, a.window, a.chunk);   // some key of the tile is seen by some row
+      const int key0 = tile_of(i) * kKeysPerTile;
+      const bool in_window = !limited || key0 < a.keep_first || key0 + 63 >= prompt_first_visible(warp_lo, a.window, a.chunk);   // some key of the tile is seen by some row
       if (key0 <= warp_hi && in_window) {
         const uint32_t k_tile = smem_u32(smem + s * STAGE_BYTES);
         float sc[8][4];
@@ -179,7 +185,7 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
         qk_tile<DH, 8, L>(sc, qf, k_tile, 0);
         // no mask where every key of the tile is at or below every row's position and inside every row's window
         const bool full_tile = !shaped && row0 + warp * 16 + 15 < rows && key0 + 63 <= warp_lo &&
-                               (!limited || key0 >= prompt_first_visible(warp_hi, a.window, a.chunk));
+                               (!limited || key0 + 63 < a.keep_first || key0 >= prompt_first_visible(warp_hi, a.window, a.chunk));
         if (full_tile) {
 #pragma unroll
           for (int j = 0; j < 8; ++j) {
@@ -193,7 +199,7 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
             for (int e = 0; e < 4; ++e) {
               const int key = key0 + j * 8 + tq * 2 + (e & 1);
               const int pos = row_pos[e >> 1];
-              const bool ok = key <= pos && key >= row_lo[e >> 1];
+              const bool ok = key <= pos && (key >= row_lo[e >> 1] || key < a.keep_first);
               float v = sc[j][e] * a.scale_log2;
               if (shaped && ok) {
                 v = sc[j][e] * scale;
@@ -218,7 +224,12 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
     for (int half = 0; half < 2; ++half) {
       const int row = row0 + warp * 16 + g + 8 * half;
       if (row >= rows) continue;
-      const float inv = l[half] > 0.0f ? 1.0f / l[half] : 0.0f;
+      float inv = l[half] > 0.0f ? 1.0f / l[half] : 0.0f;
+      if (a.sink != nullptr && l[half] > 0.0f) {
+        const float sink = a.sink[kvh * G + row % G] * 1.4426950408889634f, top = fmaxf(m[half], sink);
+        const float rescale = exp2f(m[half] - top);
+        inv = rescale / fmaf(l[half], rescale, exp2f(sink - top));
+      }
       const long long at = ((static_cast<long long>(t0 + row / G) * a.q_heads + kvh * G + row % G) * v_slices + v_slice) * DH;
       if (a.out_f32) {
         float* o = reinterpret_cast<float*>(a.out) + at;
@@ -271,7 +282,8 @@ static int prompt_tma(const void* q, long long q_stride, const void* k_cache, co
                       const int* query_start, const int* context_lens, const int* block_tables, int max_blocks, int n_seqs,
                       int max_queries, int q_heads, int kv_heads, int head_dim, int page_size, int pages, int window,
                       float scale, int exact_weights, cudaStream_t s, int cache_heads = 0, int k_ld = 0, int v_ld = 0, int v_shift = 0,
-                      int chunk = 0, float softcap = 0.0f, const float* r1 = nullptr, const float* r2 = nullptr, int out_f32 = 0) {
+                      int chunk = 0, float softcap = 0.0f, const float* r1 = nullptr, const float* r2 = nullptr, int out_f32 = 0,
+                      int keep_first = 0, const float* sink = nullptr) {
   TIE_REQUIRE(head_dim == 64 || head_dim == 128 || head_dim == 256, "attention_prompt: head_dim %d is not 64, 128 or 256", head_dim);
   TIE_REQUIRE(q_heads > 0 && kv_heads > 0 && q_heads % kv_heads == 0 && q_heads / kv_heads <= 16,
               "attention_prompt: %d query heads over %d kv heads (at most 16 per group)", q_heads, kv_heads);
@@ -296,7 +308,7 @@ static int prompt_tma(const void* q, long long q_stride, const void* k_cache, co
   TIE_REQUIRE(status_word() != nullptr, "attention_prompt: cannot allocate the status word");
   PromptArgs a{static_cast<const __nv_bfloat16*>(q), static_cast<__nv_bfloat16*>(out), query_start, context_lens, block_tables,
                status_word(), q_stride, max_blocks, q_heads, kv_heads, page_size, shift, window, scale * 1.4426950408889634f,
-               exact_weights, cache_heads, k_ld, v_ld, v_shift, chunk, softcap, r1, r2, out_f32};
+               exact_weights, cache_heads, k_ld, v_ld, v_shift, chunk, softcap, r1, r2, out_f32, keep_first, sink};
   const int max_rows = max_queries * (q_heads / kv_heads);
   int st = kOk;
   if (head_dim == 64) st = launch_prompt_tma<64>(km, vm, a, n_seqs, max_rows, s);
@@ -336,4 +348,16 @@ TIE_API int tie_attention_prompt_maps(const void* q, long long q_stride, const v
   return prompt_tma(q, q_stride, k_cache, v_cache, out, query_start, context_lens, block_tables, max_blocks, n_seqs, max_queries,
                     q_heads, kv_heads, head_dim, page_size, pages, window, scale, 1, s, cache_heads, k_ld, v_ld, v_shift, chunk, softcap,
                     r1, r2, 1);
+}
+
+// A window beside which the sequence's first keys stay visible, capped scores (softcap, 0: none) and a sink per head (null:
+// none), with the softmax weights kept to 16 bits of mantissa; out is bfloat16 [T, q_heads * head_dim].
+TIE_API int tie_attention_prompt_kept(const void* q, long long q_stride, const void* k_cache, const void* v_cache, void* out,
+                                      const int* query_start, const int* context_lens, const int* block_tables, int max_blocks,
+                                      int n_seqs, int max_queries, int q_heads, int kv_heads, int head_dim, int page_size, int pages,
+                                      int window, int keep_first, float scale, float softcap, const float* sink, cudaStream_t s) {
+  TIE_REQUIRE(keep_first >= 0 && softcap >= 0.0f, "attention_prompt: %d kept keys, a cap of %g", keep_first, static_cast<double>(softcap));
+  return prompt_tma(q, q_stride, k_cache, v_cache, out, query_start, context_lens, block_tables, max_blocks, n_seqs, max_queries,
+                    q_heads, kv_heads, head_dim, page_size, pages, window, scale, 1, s, 0, 0, 0, 0, 0, softcap, nullptr, nullptr, 0,
+                    keep_first, sink);
 }

@@ -53,12 +53,20 @@ struct AttnArgs {
   const float* r2;
   int out_f32;              // the output rows are float whatever the storage type
   int group;                // > 0: query head h reads cached head (h / group) % kv_heads (query heads laid out map by map)
+  int keep_first;           // the sequence's first keys that stay visible beside a window
+  const float* sink;        // [q_heads] or null: exp(sink[h]) is one more term of the softmax's denominator, without a value
 };
 
-// The first key that position `pos` sees.
-__device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
-  if (chunk > 0) return pos / chunk * chunk;
-  return window > 0 ? max(0, pos - window + 1) : 0;
+// The keys that a position sees, numbered without a gap: numbers `first` .. the position itself. From `edge` on (the window's
+// first key) a number is its key; the numbers below are the kept first keys, number - first.
+struct Visible {
+  int first, edge;
+  __device__ __forceinline__ int key(int number) const { return number < edge ? number - first : number; }
+};
+
+__device__ __forceinline__ Visible visible_from(int pos, int window, int chunk, int keep_first) {
+  const int lo = chunk > 0 ? pos / chunk * chunk : (window > 0 ? max(0, pos - window + 1) : 0);
+  return Visible{lo - min(lo, keep_first), lo};
 }
 
 // What a score passes on its way to the softmax beside the scale: a cap and a bias that grows with the distance.
@@ -67,15 +75,15 @@ struct ScoreShape {
   int pos;                  // the query's position
 };
 
-// One warp: online softmax over keys [lo, hi] of one (query vector, kv head).
+// One warp: online softmax over the visible keys of numbers [lo, hi] of one (query vector, kv head).
 // q is in shared memory (float, already multiplied by nothing: scale is applied to the score).
 // Lane `l` owns output dims [l * DPL, (l + 1) * DPL). Returns m, l and acc in registers.
 template <typename T, int DPL>
 __device__ __forceinline__ void attend_range(const float* __restrict__ qs, const T* __restrict__ kc,
                                              const T* __restrict__ vc, const int* __restrict__ table, int kvh,
                                              int kv_heads, int head_dim, int v_dim, int v_ld, int page_size, float scale,
-                                             int lo, int hi, float& m, float& l, float (&acc)[DPL], int k_ld = 0, int k_off = 0,
-                                             const ScoreShape shape = ScoreShape{0.0f, 0.0f, 0.0f, 0}) {
+                                             int lo, int hi, const Visible vis, float& m, float& l, float (&acc)[DPL], int k_ld,
+                                             int k_off, const ScoreShape shape) {
   if (k_ld == 0) k_ld = head_dim;
   // whole pieces of four value elements a lane, each on its own boundary
   const bool v_quads = DPL % 4 == 0 && v_dim % DPL == 0 && v_ld % 4 == 0 && reinterpret_cast<uintptr_t>(vc) % (4 * sizeof(T)) == 0;
@@ -83,8 +91,8 @@ __device__ __forceinline__ void attend_range(const float* __restrict__ qs, const
   const int lane = threadIdx.x & 31;
   const int d0 = lane * DPL;
   for (int base = lo; base <= hi; base += 32) {
-    const int j = base + lane;
-    const bool valid = j <= hi;
+    const bool valid = base + lane <= hi;
+    const int j = vis.key(base + lane);
     int row = 0;  // index of the key's row: head_dim elements in the key plane, v_dim in the value plane
     float s = -INFINITY;
     if (valid) {
@@ -172,7 +180,7 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(AttnArgs a) {
   const int s = a.seq_of_row[t];
   const int qs0 = a.query_start[s], qs1 = a.query_start[s + 1];
   const int pos = a.context_lens[s] - (qs1 - qs0) + (t - qs0);
-  const int lo = first_visible(pos, a.window, a.chunk);
+  const Visible vis = visible_from(pos, a.window, a.chunk, a.keep_first);
   const int kvh = kv_head_of(a, h);
 
   float* qs = smem + warp * a.head_dim;
@@ -183,12 +191,18 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(AttnArgs a) {
   float m = -INFINITY, l = 0.0f, acc[DPL] = {};
   attend_range<T, DPL>(qs, static_cast<const T*>(a.k_cache), static_cast<const T*>(a.v_cache),
                        a.block_tables + static_cast<long long>(s) * a.max_blocks, kvh, a.kv_heads, a.head_dim,
-                       a.v_dim, a.v_ld ? a.v_ld : a.v_dim, a.page_size, a.scale, lo, pos, m, l, acc, a.k_ld, key_offset(a, h),
+                       a.v_dim, a.v_ld ? a.v_ld : a.v_dim, a.page_size, a.scale, vis.first, pos, vis, m, l, acc, a.k_ld, key_offset(a, h),
                        score_shape(a, h, pos));
   const int d0 = lane * DPL;
+  float rescale = 1.0f;                     // the sums as they are, or brought to the larger of their maximum and the sink
+  if (a.sink != nullptr && l > 0.0f) {
+    const float top = fmaxf(m, a.sink[h]);
+    rescale = expf(m - top);
+    l = fmaf(l, rescale, expf(a.sink[h] - top));
+  }
   if (d0 < a.v_dim) {
     const long long at = (static_cast<long long>(t) * a.q_heads + h) * a.v_dim + d0;
-    const float inv = l > 0.0f ? 1.0f / l : 0.0f;  // no keys (a padding row): zeros
+    const float inv = l > 0.0f ? rescale / l : 0.0f;  // no keys (a padding row): zeros
 #pragma unroll
     for (int e = 0; e < DPL; ++e)
       if (d0 + e < a.v_dim) {
@@ -214,8 +228,8 @@ __global__ void __launch_bounds__(128) attention_split_kernel(AttnArgs a, const 
   const int s = seq_list[li];
   const int t = a.query_start[s];
   const int pos = a.context_lens[s] - 1;
-  const int lo0 = first_visible(pos, a.window, a.chunk);
-  const int lo = lo0 + split * split_keys;
+  const Visible vis = visible_from(pos, a.window, a.chunk, a.keep_first);
+  const int lo = vis.first + split * split_keys;
   if (lo > pos) return;  // this sequence has fewer splits
   // The last split takes whatever is left, so that a context longer than max_splits * split_keys (a caller
   // who sized max_splits from something else than the longest context) costs time, never keys.
@@ -230,7 +244,7 @@ __global__ void __launch_bounds__(128) attention_split_kernel(AttnArgs a, const 
   float m = -INFINITY, l = 0.0f, acc[DPL] = {};
   attend_range<T, DPL>(qs, static_cast<const T*>(a.k_cache), static_cast<const T*>(a.v_cache),
                        a.block_tables + static_cast<long long>(s) * a.max_blocks, kvh, a.kv_heads, a.head_dim,
-                       a.v_dim, a.v_ld ? a.v_ld : a.v_dim, a.page_size, a.scale, lo, hi, m, l, acc, a.k_ld, key_offset(a, h),
+                       a.v_dim, a.v_ld ? a.v_ld : a.v_dim, a.page_size, a.scale, lo, hi, vis, m, l, acc, a.k_ld, key_offset(a, h),
                        score_shape(a, h, pos));
   float* dst = scratch + ((static_cast<long long>(li) * a.q_heads + h) * max_splits + split) * (a.v_dim + 2);
   const int d0 = lane * DPL;
@@ -275,8 +289,8 @@ __global__ void __launch_bounds__(1024) attention_group_split_kernel(AttnArgs a,
   const int s = seq_list[li];
   const int t = a.query_start[s];
   const int pos = a.context_lens[s] - 1;
-  const int lo0 = first_visible(pos, a.window, a.chunk);
-  const int lo = lo0 + split * split_keys;
+  const Visible vis = visible_from(pos, a.window, a.chunk, a.keep_first);
+  const int lo = vis.first + split * split_keys;
   if (lo > pos) return;                      // the whole block: this sequence has fewer splits
   const int hi = split == max_splits - 1 ? pos : min(pos, lo + split_keys - 1);
   // the warp's query head: the heads h with (h / group) % kv_heads == c, in order
@@ -299,8 +313,8 @@ __global__ void __launch_bounds__(1024) attention_group_split_kernel(AttnArgs a,
   for (int base = lo; base <= hi; base += kGroupTile) {
     __syncthreads();                          // everyone is through with the tile before
     if (threadIdx.x < kGroupTile) {
-      const int j = base + threadIdx.x;
-      rows[threadIdx.x] = j <= hi ? (table[j / a.page_size] * a.kv_heads + c) * a.page_size + j % a.page_size : -1;
+      const int j = vis.key(base + threadIdx.x);
+      rows[threadIdx.x] = base + static_cast<int>(threadIdx.x) <= hi ? (table[j / a.page_size] * a.kv_heads + c) * a.page_size + j % a.page_size : -1;
     }
     __syncthreads();
     if (k_vec) {
@@ -331,8 +345,8 @@ __global__ void __launch_bounds__(1024) attention_group_split_kernel(AttnArgs a,
     }
     asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory");      // the copies of this thread; the barrier does the rest
     __syncthreads();
-    const int j = base + lane;
-    const bool valid = j <= hi;
+    const int j = vis.key(base + lane);
+    const bool valid = base + lane <= hi;
     float sc = -INFINITY;
     if (valid) {
       const T* kr = k_tile + lane * k_row + k_off;
@@ -454,14 +468,15 @@ __global__ void __launch_bounds__(kMergeThreads) attention_merge_kernel(AttnArgs
     }
     return;
   }
-  const int lo0 = first_visible(pos, a.window, a.chunk);
-  const int splits = min((pos - lo0) / split_keys + 1, max_splits);   // the last one took the rest (split kernels)
+  const Visible vis = visible_from(pos, a.window, a.chunk, a.keep_first);
+  const int splits = min((pos - vis.first) / split_keys + 1, max_splits);   // the last one took the rest (split kernels)
   const int stride = a.head_dim + 2;
   const float* src = scratch + (static_cast<long long>(li) * a.q_heads + h) * max_splits * stride;
   if (threadIdx.x < 32) {
     float m = -INFINITY;
     for (int i = threadIdx.x; i < splits; i += 32) m = fmaxf(m, src[i * stride + a.head_dim]);
     m = warp_max(m);
+    if (a.sink != nullptr) m = fmaxf(m, a.sink[h]);
     float l = 0.0f;
     for (int i = threadIdx.x; i < splits; i += 32) {
       const float w = expf(src[i * stride + a.head_dim] - m);
@@ -469,6 +484,7 @@ __global__ void __launch_bounds__(kMergeThreads) attention_merge_kernel(AttnArgs
       l += src[i * stride + a.head_dim + 1] * w;   // summed below in a fixed lane order
     }
     l = warp_sum(l);
+    if (a.sink != nullptr) l += expf(a.sink[h] - m);
     if (threadIdx.x == 0) inv_l = l > 0.0f ? 1.0f / l : 0.0f;
   }
   __syncthreads();
@@ -683,6 +699,45 @@ TIE_API int tie_attention_maps_split(int dtype, const void* q, long long q_strid
   if (dtype == TIE_F32) return launch_attention<float>(a, nullptr, seq_list, n_list, split_keys, max_splits, scratch, 0, s, true);
   if (dtype == TIE_BF16)
     return launch_attention<__nv_bfloat16>(a, nullptr, seq_list, n_list, split_keys, max_splits, scratch, 0, s, true);
+  set_error("attention: unknown dtype code %d", dtype);
+  return kBadArgument;
+}
+
+// A window of keys beside which the sequence's first keys stay visible (keep_first), capped scores (softcap, 0: none) and a
+// sink per head (null: none), for keys and values of any two sizes: all rows of the step's first `rows`, or one row per
+// listed sequence with its visible keys in splits.
+TIE_API int tie_attention_kept_rows(int dtype, const void* q, long long q_stride, const void* k_cache, const void* v_cache,
+                                    void* out, const int* seq_of_row, const int* query_start, const int* context_lens,
+                                    const int* block_tables, int max_blocks, int rows, int seqs, int q_heads, int kv_heads,
+                                    int head_dim, int v_dim, int page_size, int window, int keep_first, float scale, float softcap,
+                                    const float* sink, cudaStream_t s) {
+  AttnArgs a{q, k_cache, v_cache, out, seq_of_row, query_start, context_lens, block_tables, q_stride, max_blocks,
+             rows, seqs, q_heads, kv_heads, head_dim, page_size, window, scale, v_dim};
+  a.softcap = softcap, a.keep_first = keep_first, a.sink = sink;
+  TIE_REQUIRE(keep_first >= 0 && softcap >= 0.0f, "attention: %d kept keys, a cap of %g", keep_first, static_cast<double>(softcap));
+  if (const int st = check_attn(a, true)) return st;
+  if (dtype == TIE_F32) return launch_attention<float>(a, nullptr, nullptr, 0, 0, 0, nullptr, 1, s);
+  if (dtype == TIE_BF16) return launch_attention<__nv_bfloat16>(a, nullptr, nullptr, 0, 0, 0, nullptr, 1, s);
+  set_error("attention: unknown dtype code %d", dtype);
+  return kBadArgument;
+}
+
+TIE_API int tie_attention_kept_split(int dtype, const void* q, long long q_stride, const void* k_cache, const void* v_cache,
+                                     void* out, const int* query_start, const int* context_lens, const int* block_tables,
+                                     int max_blocks, int seqs, int q_heads, int kv_heads, int head_dim, int v_dim, int page_size,
+                                     int window, int keep_first, float scale, float softcap, const float* sink, const int* seq_list,
+                                     int n_list, int split_keys, int max_splits, float* scratch, cudaStream_t s) {
+  AttnArgs a{q, k_cache, v_cache, out, nullptr, query_start, context_lens, block_tables, q_stride, max_blocks,
+             0, seqs, q_heads, kv_heads, head_dim, page_size, window, scale, v_dim};
+  a.softcap = softcap, a.keep_first = keep_first, a.sink = sink;
+  TIE_REQUIRE(keep_first >= 0 && softcap >= 0.0f, "attention: %d kept keys, a cap of %g", keep_first, static_cast<double>(softcap));
+  if (const int st = check_attn(a, true)) return st;
+  TIE_REQUIRE(split_keys > 0 && max_splits > 0 && max_splits <= kMergeMaxSplits && scratch != nullptr,
+              "attention split: bad split geometry (at most %d splits)", kMergeMaxSplits);
+  const bool grouped = q_heads > kv_heads;      // heads that share keys: one block reads them once for all of them
+  if (dtype == TIE_F32) return launch_attention<float>(a, nullptr, seq_list, n_list, split_keys, max_splits, scratch, 0, s, grouped);
+  if (dtype == TIE_BF16)
+    return launch_attention<__nv_bfloat16>(a, nullptr, seq_list, n_list, split_keys, max_splits, scratch, 0, s, grouped);
   set_error("attention: unknown dtype code %d", dtype);
   return kBadArgument;
 }

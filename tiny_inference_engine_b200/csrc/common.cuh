@@ -110,6 +110,9 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   return scratch[32];
 }
 
+// The activation of a gated product's epilogue: 1 the SiLU, 2 the ReLU.
+__device__ __forceinline__ float gate_act(float g, int act) { return act == 2 ? fmaxf(g, 0.0f) : g / (1.0f + expf(-g)); }
+
 inline int ceil_div(long long a, long long b) { return static_cast<int>((a + b - 1) / b); }
 
 // Programmatic dependent launch. Every kernel of this library starts with pdl_sync(): it waits

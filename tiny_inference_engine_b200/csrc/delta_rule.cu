@@ -168,8 +168,8 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
   // A buffer: k [chunk][dim], q [chunk][dim], decays [chunk][dim], v [chunk][kDeltaCols], beta [chunk].
   const int buf_floats = (chunk * (3 * dim + kDeltaCols + 1) + 3) & ~3;      // a buffer starts on a 16-byte boundary
   const bool vec4 = dim % 4 == 0;
-  const bool wide = !decay_per_head && vec4 && nqk % 4 == 0 && decay_stride % 4 == 0 && ((reinterpret_cast<uintptr_t>(kn) | reinterpret_cast<uintptr_t>(qn) |
-                                                                      reinterpret_cast<uintptr_t>(decay)) & 15) == 0;
+  const bool wide = vec4 && nqk % 4 == 0 && ((reinterpret_cast<uintptr_t>(kn) | reinterpret_cast<uintptr_t>(qn)) & 15) == 0 &&
+                    (decay_per_head || (decay_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(decay) & 15) == 0));
   auto fetch = [&](int c0, float* base) {
     const int cn = min(chunk, n - c0);
     float* kb = base;
@@ -184,7 +184,7 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
         const long long t = t0 + c0 + tc;
         async_copy16(kb + tc * dim + d, kn + t * nqk + g * dim + d);
         async_copy16(qb + tc * dim + d, qn + t * nqk + g * dim + d);
-        async_copy16(gb + tc * dim + d, decay + t * decay_stride + h * dim + d);
+        if (!decay_per_head) async_copy16(gb + tc * dim + d, decay + t * decay_stride + h * dim + d);
       }
     } else {
       for (int i = threadIdx.x; i < cn * dim; i += blockDim.x) {
@@ -192,7 +192,7 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
         const long long t = t0 + c0 + tc;
         async_copy4(kb + i, kn + t * nqk + g * dim + d);
         async_copy4(qb + i, qn + t * nqk + g * dim + d);
-        async_copy4(gb + i, decay + t * decay_stride + (decay_per_head ? h : h * dim + d));
+        if (!decay_per_head) async_copy4(gb + i, decay + t * decay_stride + h * dim + d);
       }
     }
     for (int i = threadIdx.x; i < cn * kDeltaCols; i += blockDim.x) {
@@ -200,6 +200,8 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
       if (c < vdim) async_copy4(vb + i, vn + (t0 + c0 + tc) * static_cast<long long>(nv) + h * vdim + c);
       else vb[i] = 0.0f;
     }
+    if (decay_per_head)                       // one factor a token and head: at the start of the token's row
+      for (int i = threadIdx.x; i < cn; i += blockDim.x) async_copy4(gb + i * dim, decay + (t0 + c0 + i) * decay_stride + h);
     for (int i = threadIdx.x; i < cn; i += blockDim.x) {
       if (beta) async_copy4(bb + i, beta + (t0 + c0 + i) * static_cast<long long>(sh.heads) + h);
       else bb[i] = 1.0f;
@@ -243,8 +245,8 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
         float kk[4], qq[4], gg[4];
         if (vec4) {                              // dim % 4 == 0: the lane's four channels are one 16-byte piece
           if (r0 < dim) {
-            const float4 k4 = *reinterpret_cast<const float4*>(kt + r0), q4v = *reinterpret_cast<const float4*>(qt + r0),
-                         g4 = *reinterpret_cast<const float4*>(gt + r0);
+            const float4 k4 = *reinterpret_cast<const float4*>(kt + r0), q4v = *reinterpret_cast<const float4*>(qt + r0);
+            const float4 g4 = decay_per_head ? make_float4(gt[0], gt[0], gt[0], gt[0]) : *reinterpret_cast<const float4*>(gt + r0);
             kk[0] = k4.x, kk[1] = k4.y, kk[2] = k4.z, kk[3] = k4.w;
             qq[0] = q4v.x, qq[1] = q4v.y, qq[2] = q4v.z, qq[3] = q4v.w;
             gg[0] = g4.x, gg[1] = g4.y, gg[2] = g4.z, gg[3] = g4.w;
@@ -258,7 +260,7 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
             const bool in = r0 + e < dim;
             kk[e] = in ? kt[r0 + e] : 0.0f;
             qq[e] = in ? qt[r0 + e] : 0.0f;
-            gg[e] = in ? gt[r0 + e] : 0.0f;
+            gg[e] = in ? gt[decay_per_head ? 0 : r0 + e] : 0.0f;
           }
         }
 #pragma unroll

@@ -19,7 +19,7 @@ namespace tie {
 // ((i / 64) * k_block_rows + id) * 64 + i % 64.
 template <typename T>
 __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ x,
-                             int dim, int vocab, int k_block_rows) {
+                             int dim, int vocab, int k_block_rows, float scale) {
   pdl_sync();
   const int t = blockIdx.x;
   int id = ids[t];
@@ -36,17 +36,17 @@ __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict_
                               : table + static_cast<size_t>(id) * dim + i);
 #pragma unroll
       for (int e = 0; e < V; e += 4)
-        *reinterpret_cast<float4*>(out + i + e) = make_float4(v.v[e], v.v[e + 1], v.v[e + 2], v.v[e + 3]);
+        *reinterpret_cast<float4*>(out + i + e) = make_float4(v.v[e] * scale, v.v[e + 1] * scale, v.v[e + 2] * scale, v.v[e + 3] * scale);
     }
     return;
   }
   if (k_block_rows > 0) {
     for (int i = threadIdx.x; i < dim; i += blockDim.x)
-      out[i] = ld(table + (static_cast<size_t>(i >> 6) * k_block_rows + id) * 64 + (i & 63));
+      out[i] = ld(table + (static_cast<size_t>(i >> 6) * k_block_rows + id) * 64 + (i & 63)) * scale;
     return;
   }
   const T* row = table + static_cast<size_t>(id) * dim;
-  for (int i = threadIdx.x; i < dim; i += blockDim.x) out[i] = ld(row + i);
+  for (int i = threadIdx.x; i < dim; i += blockDim.x) out[i] = ld(row + i) * scale;
 }
 
 // tokens[dst[i]] = ids[src[i]]: a step that is queued before the host has seen the ids sampled by the step ahead
@@ -599,9 +599,9 @@ __global__ void __launch_bounds__(256, 4) qk_norm_rope_append_rows_kernel(T* __r
 
 // ---------------------------------------------------------------------------------------------
 template <typename T>
-int launch_embed(const void* table, const int* ids, float* x, int tokens, int dim, int vocab, int k_block_rows, cudaStream_t s) {
+int launch_embed(const void* table, const int* ids, float* x, int tokens, int dim, int vocab, int k_block_rows, float scale, cudaStream_t s) {
   if (tokens == 0) return kOk;
-  TIE_LAUNCH((embed_kernel<T>), tokens, dim >= 1024 ? 256 : 128, 0, s, static_cast<const T*>(table), ids, x, dim, vocab, k_block_rows);
+  TIE_LAUNCH((embed_kernel<T>), tokens, dim >= 1024 ? 256 : 128, 0, s, static_cast<const T*>(table), ids, x, dim, vocab, k_block_rows, scale);
   TIE_RETURN_LAUNCH("embed");
 }
 
@@ -753,13 +753,14 @@ using namespace tie;
     return kBadArgument;                                               \
   } while (0)
 
-// k_block_rows > 0: the table is stored in k-blocks of 64 columns, k_block_rows rows each (see embed_kernel).
+// k_block_rows > 0: the table is stored in k-blocks of 64 columns, k_block_rows rows each (see embed_kernel). Rows are
+// multiplied by `scale` in float.
 TIE_API int tie_embed(int dtype, const void* table, const int* ids, float* x, int tokens, int dim, int vocab,
-                      int k_block_rows, cudaStream_t s) {
+                      int k_block_rows, float scale, cudaStream_t s) {
   TIE_REQUIRE(tokens >= 0 && dim > 0 && vocab > 0 && (k_block_rows == 0 || k_block_rows >= vocab),
               "embed: bad sizes tokens=%d dim=%d vocab=%d (k-blocks of %d rows)", tokens, dim, vocab, k_block_rows);
-  TIE_DISPATCH(dtype, launch_embed<float>(table, ids, x, tokens, dim, vocab, k_block_rows, s),
-               launch_embed<__nv_bfloat16>(table, ids, x, tokens, dim, vocab, k_block_rows, s));
+  TIE_DISPATCH(dtype, launch_embed<float>(table, ids, x, tokens, dim, vocab, k_block_rows, scale, s),
+               launch_embed<__nv_bfloat16>(table, ids, x, tokens, dim, vocab, k_block_rows, scale, s));
 }
 
 TIE_API int tie_scatter_ids(int* tokens, const int* dst, const int* src, const int* ids, int n, cudaStream_t s) {

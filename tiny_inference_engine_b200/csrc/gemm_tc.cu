@@ -230,7 +230,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
       const int i = i0 + warp * 32 + lane;
       if (silu) {
         // The weight rows come in blocks of 16 gate rows followed by their 16 up rows; the output is
-        // silu(gate) * up, half as wide as the product: out[token, 16 * block + r].
+        // act(gate) * up (act 1: the SiLU, 2: the ReLU), half as wide as the product: out[token, 16 * block + r].
         if (transposed) {
           // lanes 0-15 of a warp hold gate rows, lanes 16-31 the matching up rows: exchange, then
           // the lower half finishes columns 0-7 of each chunk and the upper half columns 8-15
@@ -250,7 +250,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
               const float g = __uint_as_float(upper ? got : r[e]);
               const float u = __uint_as_float(upper ? r[e + 8] : got);
               const int j = j0 + c0 + e + (upper ? 8 : 0);
-              if (j < rows_y && o < (rows_x >> 1)) st(out + static_cast<long long>(j) * ldo + o, g / (1.0f + expf(-g)) * u);
+              if (j < rows_y && o < (rows_x >> 1)) st(out + static_cast<long long>(j) * ldo + o, gate_act(g, silu) * u);
             }
           }
         } else {
@@ -266,7 +266,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
 #pragma unroll
               for (int e = 0; e < 16; ++e) {
                 const float gv = __uint_as_float(g[e]);
-                v[e] = gv / (1.0f + expf(-gv)) * __uint_as_float(u[e]);
+                v[e] = gate_act(gv, silu) * __uint_as_float(u[e]);
               }
               const long long at = static_cast<long long>(i) * ldo + ((j0 + c0) >> 1);
               if (((at * sizeof(OutT)) & 15) == 0 && sizeof(OutT) == 2) {
@@ -409,7 +409,7 @@ using namespace tie;
 // with tie_gemm_tc_scratch_floats floats: the float partial sums [splits, M, N]; with reduce == 0
 // they are left there for a consumer that adds them itself (tie_gemm_tc_real_splits says how
 // many there are). silu != 0: w holds blocks of 16 gate rows followed by their 16 up rows and
-// out[M, N / 2] = silu(gate) * up. deep != 0: the deepest shared-memory ring (one CTA per SM), else
+// out[M, N / 2] = act(gate) * up, act the SiLU (1) or the ReLU (2). deep != 0: the deepest shared-memory ring (one CTA per SM), else
 // a ring of about 100 KB (two CTAs per SM). Returns kBadArgument
 // with a message for sizes it does not take (K or a row stride not a multiple of 8, unaligned
 // pointers): the caller then uses the CUDA-core kernel.

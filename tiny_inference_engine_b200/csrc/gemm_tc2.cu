@@ -228,7 +228,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
 #pragma unroll
             for (int e = 0; e < 16; ++e) {
               const float gv = __uint_as_float(g[e]);
-              v[e] = gv / (1.0f + expf(-gv)) * __uint_as_float(u[e]);
+              v[e] = gate_act(gv, silu) * __uint_as_float(u[e]);
             }
             const long long at = static_cast<long long>(i) * ldo + ((j0 + c0) >> 1);
             if (((at * sizeof(OutT)) & 15) == 0 && sizeof(OutT) == 2) {
@@ -375,7 +375,7 @@ static int launch_tc2(const CUtensorMap& ma, const CUtensorMap& mw, void* out, i
 
 using namespace tie;
 
-// out[M, N] (or, with silu, out[M, N / 2] = silu(gate) * up for w in blocks of 16 gate + 16 up rows)
+// out[M, N] (or, with silu 1 or 2, out[M, N / 2] = act(gate) * up, act the SiLU or the ReLU, for w in blocks of 16 gate + 16 up rows)
 // = a[M, K] . w[N, K]^T on pairs of SMs. a, w bfloat16 with K and row strides multiples of 8. w_rows > 0: w is
 // stored in k-blocks, [ceil(K / 64)][w_rows][64], and the product uses its rows w_row0 .. w_row0 + N - 1 (gemm_tc.cu).
 // How many pairs of SMs hold the kernel at once: what the host counts waves of tiles with.

@@ -241,6 +241,15 @@ __global__ void scale_rows_kernel(float* __restrict__ x, long long stride, int w
   x[(i / width) * stride + i % width] *= c;
 }
 
+__global__ void cap_rows_kernel(float* __restrict__ x, long long stride, int width, long long total, float cap) {
+  pdl_sync();
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    float* p = x + (i / width) * stride + i % width;
+    *p = cap * tanhf(*p / cap);
+  }
+}
+
 template <typename T>
 int launch_add_normed_rmsnorm(float* x, const void* delta, const float* part, long long part_stride, int splits,
                               const float* bias, const float* wb, float eps_b, float mult, const int* rows,
@@ -373,4 +382,14 @@ TIE_API int tie_scale_rows(float* x, long long stride, int rows, int width, floa
   if (total == 0) return kOk;
   TIE_LAUNCH(scale_rows_kernel, ceil_div(total, 256), 256, 0, s, x, stride, width, total, c);
   TIE_RETURN_LAUNCH("scale_rows");
+}
+
+// x = cap * tanh(x / cap) for float rows, in place.
+TIE_API int tie_cap_rows(float* x, long long stride, int rows, int width, float cap, cudaStream_t s) {
+  TIE_REQUIRE(rows >= 0 && width > 0 && cap > 0.0f, "cap_rows: bad sizes rows=%d width=%d cap=%g", rows, width, static_cast<double>(cap));
+  const long long total = static_cast<long long>(rows) * width;
+  if (total == 0) return kOk;
+  const int blocks = static_cast<int>(min(static_cast<long long>(148 * 8), (total + 255) / 256));
+  TIE_LAUNCH(cap_rows_kernel, blocks, 256, 0, s, x, stride, width, total, cap);
+  TIE_RETURN_LAUNCH("cap_rows");
 }

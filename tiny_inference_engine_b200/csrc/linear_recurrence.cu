@@ -10,6 +10,7 @@
 //
 // Kernels (float inside; T is the storage type of the projections and of the outputs that feed a product):
 //   gla_prep      one block per token.
+//   act_split     q, k, v behind an activation as float rows (linear attention with constant decays).
 //   ssd_prep      one block per (token, unit): units are the heads of C, of B and of x, and one for the step sizes.
 //                 The convolution's first taps - 1 inputs come from the rows ahead in the step or from the tail that
 //                 the sequence's state slot keeps behind S (channels in the order C, B, x).
@@ -41,6 +42,50 @@ __global__ void __launch_bounds__(256) gla_prep_kernel(const T* __restrict__ pro
     *a = expf(-lr_softplus(-z) * inv_tau);
   }
   for (int c = threadIdx.x; c < nv; c += blockDim.x) vn[t * nv + c] = ld(row + v_off + c);
+}
+
+// q, k and v behind an activation (1: the SiLU), as float rows.
+template <typename T>
+__global__ void __launch_bounds__(256) act_split_kernel(const T* __restrict__ proj, long long stride, int q_off, int k_off, int v_off,
+                                                        int nqk, int nv, int act, float* __restrict__ qn, float* __restrict__ kn,
+                                                        float* __restrict__ vn, long long total) {
+  pdl_sync();
+  const int width = 2 * nqk + nv;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long t = i / width;
+    const int c = static_cast<int>(i - t * width);
+    const int at = c < nqk ? q_off + c : (c < 2 * nqk ? k_off + c - nqk : v_off + c - 2 * nqk);
+    const float z = ld(proj + t * stride + at);
+    float* dst = c < nqk ? qn + t * nqk + c : (c < 2 * nqk ? kn + t * nqk + c - nqk : vn + t * nv + c - 2 * nqk);
+    *dst = act == 1 ? z * lr_sigmoid(z) : z;
+  }
+}
+
+// The same, 16 bytes of the projection a thread: sections and sizes in whole vectors.
+template <typename T>
+__global__ void __launch_bounds__(256) act_split_vec_kernel(const T* __restrict__ proj, long long stride, int q_off, int k_off, int v_off,
+                                                            int nqk, int nv, int act, float* __restrict__ qn, float* __restrict__ kn,
+                                                            float* __restrict__ vn, long long total) {
+  pdl_sync();
+  constexpr int V = Vec16<T>::N;
+  const int pieces = (2 * nqk + nv) / V;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long t = i / pieces;
+    const int c = static_cast<int>(i - t * pieces) * V;
+    const int at = c < nqk ? q_off + c : (c < 2 * nqk ? k_off + c - nqk : v_off + c - 2 * nqk);
+    float* dst = c < nqk ? qn + t * nqk + c : (c < 2 * nqk ? kn + t * nqk + c - nqk : vn + t * nv + c - 2 * nqk);
+    Vec16<T> z;
+    z.load(proj + t * stride + at);
+#pragma unroll
+    for (int e = 0; e < V; e += 4) {
+      float o[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) o[k] = act == 1 ? z.v[e + k] * lr_sigmoid(z.v[e + k]) : z.v[e + k];
+      store4(dst + e, o);
+    }
+  }
 }
 
 struct SsdShape {
@@ -121,6 +166,26 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* __rest
   }
 }
 
+// The same for long heads (or one norm over a whole row): one block per (token, head).
+template <typename T>
+__global__ void __launch_bounds__(256) head_norm_gate_block_kernel(const float* __restrict__ o, const T* __restrict__ gate,
+                                                                   long long gate_stride, const float* __restrict__ w, float eps,
+                                                                   T* __restrict__ out, int heads, int vdim, int act) {
+  pdl_sync();
+  __shared__ float scratch[33];
+  const long long item = blockIdx.x, t = item / heads;
+  const int h = static_cast<int>(item % heads);
+  const float* x = o + item * vdim;
+  float ss = 0.0f;
+  for (int d = threadIdx.x; d < vdim; d += blockDim.x) ss += x[d] * x[d];
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(vdim) + eps);
+  for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
+    const float g = ld(gate + t * gate_stride + h * vdim + d);
+    const float a = act == 1 ? g * lr_sigmoid(g) : lr_sigmoid(g);
+    st(out + item * vdim + d, ((x[d] * inv) * w[d]) * a);
+  }
+}
+
 // y = (o + skip[h] x) * silu(z), each of `parts` equal parts of the row divided by its own root mean square, times w.
 template <typename T>
 __global__ void __launch_bounds__(256) ssd_out_kernel(const float* __restrict__ o, const float* __restrict__ xn,
@@ -177,6 +242,26 @@ TIE_API int tie_gla_prep(int dtype, const void* proj, long long stride, int q_of
   TIE_RETURN_LAUNCH("gla_prep");
 }
 
+TIE_API int tie_act_split(int dtype, const void* proj, long long stride, int q_off, int k_off, int v_off, int tokens, int nqk, int nv,
+                          int act, float* qn, float* kn, float* vn, cudaStream_t s) {
+  TIE_REQUIRE(nqk > 0 && nv > 0 && (act == 0 || act == 1), "act_split: bad sizes nqk=%d nv=%d act=%d", nqk, nv, act);
+  if (tokens <= 0) return kOk;
+  const int vec = dtype == TIE_F32 ? 4 : 8;
+  auto on16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const bool wide = on16(proj) && on16(qn) && on16(kn) && on16(vn) && stride % vec == 0 && q_off % vec == 0 && k_off % vec == 0 &&
+                    v_off % vec == 0 && nqk % vec == 0 && nv % vec == 0;
+  const long long total = static_cast<long long>(tokens) * (2 * nqk + nv) / (wide ? vec : 1);
+  const int blocks = static_cast<int>(min(static_cast<long long>(148 * 8), (total + 255) / 256));
+  if (wide) {
+    TIE_BY_DTYPE(dtype, TIE_LAUNCH((act_split_vec_kernel<T>), blocks, 256, 0, s, static_cast<const T*>(proj), stride, q_off, k_off, v_off,
+                                   nqk, nv, act, qn, kn, vn, total));
+  } else {
+    TIE_BY_DTYPE(dtype, TIE_LAUNCH((act_split_kernel<T>), blocks, 256, 0, s, static_cast<const T*>(proj), stride, q_off, k_off, v_off, nqk,
+                                   nv, act, qn, kn, vn, total));
+  }
+  TIE_RETURN_LAUNCH("act_split");
+}
+
 TIE_API int tie_ssd_prep(int dtype, const void* proj, long long stride, int c_off, int b_off, int x_off, int dt_off,
                          const float* conv_w, const float* conv_b, const float* state, long long state_stride,
                          long long conv_state_off, const int* seq_of_row, const int* query_start, const int* state_slots,
@@ -200,6 +285,11 @@ TIE_API int tie_head_norm_gate(int dtype, const float* o, const void* gate, long
               tokens, heads, vdim, act);
   const long long items = static_cast<long long>(tokens) * heads;
   if (items == 0) return kOk;
+  if (vdim >= 512 && items <= 0x7fffffffLL) {
+    TIE_BY_DTYPE(dtype, TIE_LAUNCH((head_norm_gate_block_kernel<T>), static_cast<int>(items), 256, 0, s, o, static_cast<const T*>(gate),
+                                   gate_stride, w, eps, static_cast<T*>(out), heads, vdim, act));
+    TIE_RETURN_LAUNCH("head_norm_gate");
+  }
   TIE_BY_DTYPE(dtype, TIE_LAUNCH((head_norm_gate_kernel<T>), ceil_div(items, 4), 128, 0, s, o, static_cast<const T*>(gate),
                                  gate_stride, w, eps, static_cast<T*>(out), heads, vdim, act, items));
   TIE_RETURN_LAUNCH("head_norm_gate");

@@ -37,14 +37,14 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 }
 
 // smem per warp: experts floats (scores), experts floats (work), groups floats, groups ints.
-// score_fn 0: s = softmax over all experts; 1: s = sigmoid of each logit. Experts are chosen by s + correction
+// score_fn 0: s = softmax over all experts; 1: s = sigmoid of each logit (logits plus `bias`, where given). Experts are chosen by s + correction
 // (correction null: by s); a group counts as the sum of its `group_top` largest choice scores (1: its best member);
 // experts outside the kept groups cannot be chosen (their choice score counts as minus infinity: choice scores may be
 // negative). The weights are the chosen experts' s, over their sum (+ 1e-20) when `renorm`, else as they are.
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, long long ld_logits, int tokens,
                                                         int experts, int top, int groups, int keep, int score_fn,
                                                         const float* __restrict__ correction, int group_top, int renorm,
-                                                        float weight_scale, int* __restrict__ ids, float* __restrict__ weights) {
+                                                        float weight_scale, const float* __restrict__ bias, int* __restrict__ ids, float* __restrict__ weights) {
   pdl_sync();
   extern __shared__ float smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -57,11 +57,11 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
   const float* z = logits + t * ld_logits;
   if (score_fn == 0) {
     float m = -INFINITY;
-    for (int e = lane; e < experts; e += 32) m = fmaxf(m, z[e]);
+    for (int e = lane; e < experts; e += 32) m = fmaxf(m, z[e] + (bias != nullptr ? bias[e] : 0.0f));
     m = warp_max(m);
     float sum = 0.0f;
     for (int e = lane; e < experts; e += 32) {
-      const float p = expf(z[e] - m);
+      const float p = expf(z[e] + (bias != nullptr ? bias[e] : 0.0f) - m);
       score[e] = p;
       sum += p;
     }
@@ -69,7 +69,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
     const float inv = 1.0f / sum;
     for (int e = lane; e < experts; e += 32) score[e] *= inv;
   } else {
-    for (int e = lane; e < experts; e += 32) score[e] = 1.0f / (1.0f + expf(-z[e]));
+    for (int e = lane; e < experts; e += 32) score[e] = 1.0f / (1.0f + expf(-(z[e] + (bias != nullptr ? bias[e] : 0.0f))));
   }
   for (int e = lane; e < experts; e += 32) work[e] = score[e] + (correction != nullptr ? correction[e] : 0.0f);
   __syncwarp();
@@ -406,7 +406,7 @@ TIE_API int tie_moe_combine(int dtype, const void* y, const int* sorted, const i
 }
 
 TIE_API int tie_moe_route(const float* logits, long long ld_logits, int tokens, int experts, int top, int groups, int keep,
-                          int score_fn, const float* correction, int group_top, int renorm, float weight_scale, int* ids,
+                          int score_fn, const float* correction, int group_top, int renorm, float weight_scale, const float* bias, int* ids,
                           float* weights, cudaStream_t s) {
   TIE_REQUIRE((score_fn == 0 || score_fn == 1) && group_top >= 1, "moe_route: score function %d, %d members a group's score",
               score_fn, group_top);
@@ -417,7 +417,7 @@ TIE_API int tie_moe_route(const float* logits, long long ld_logits, int tokens, 
   const size_t smem = 4 * sizeof(float) * (2 * experts + 2 * groups);
   TIE_REQUIRE(smem <= 48 * 1024, "moe_route: %d experts exceed the kernel's shared memory", experts);
   TIE_LAUNCH(moe_route_kernel, ceil_div(tokens, 4), 128, smem, s, logits, ld_logits, tokens, experts, top, groups, keep, score_fn,
-             correction, group_top, renorm, weight_scale, ids, weights);
+             correction, group_top, renorm, weight_scale, bias, ids, weights);
   TIE_RETURN_LAUNCH("moe_route");
 }
 

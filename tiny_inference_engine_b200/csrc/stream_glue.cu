@@ -3,7 +3,7 @@
 //   add_concat   x += delta (a tensor, or the partial sums of a split product added in order), then
 //                out[t] = [x[t] | other[t]] in the storage type: the input of a product over the stream and a second
 //                stream side by side (a model that mixes its embedding back in ahead of a span of layers).
-//   glu_biased   out[t, i] = act(g[t, i] + bg[i]) * (u[t, i] + bu[i]), act the SiLU or the tanh form of GELU; out may be
+//   glu_biased   out[t, i] = act(g[t, i] + bg[i]) * (u[t, i] + bu[i]), act the SiLU, the tanh form of GELU or the ReLU; out may be
 //                wider than the unit: column I is then 1 and the columns after it 0, so that a product over
 //                [W_down | bias | 0] adds the bias inside its float accumulator.
 #include <math.h>
@@ -52,7 +52,7 @@ __global__ void glu_biased_kernel(const T* __restrict__ gu, const float* __restr
   }
   const float g = ld(gu + t * 2 * inter + i) + (bg ? bg[i] : 0.0f);
   const float u = ld(gu + t * 2 * inter + inter + i) + (bu ? bu[i] : 0.0f);
-  const float a = act == 1 ? gelu_tanh_f(g) : g / (1.0f + expf(-g));
+  const float a = act == 1 ? gelu_tanh_f(g) : (act == 2 ? fmaxf(g, 0.0f) : g / (1.0f + expf(-g)));
   st(out + idx, a * u);
 }
 
@@ -78,7 +78,7 @@ __global__ void glu_biased_vec_kernel(const T* __restrict__ gu, const float* __r
 #pragma unroll
     for (int j = 0; j < V; ++j) {
       const float gv = g.v[j] + (bg ? bg[i + j] : 0.0f), uv = u.v[j] + (bu ? bu[i + j] : 0.0f);
-      o.v[j] = (act == 1 ? gelu_tanh_f(gv) : gv / (1.0f + expf(-gv))) * uv;
+      o.v[j] = (act == 1 ? gelu_tanh_f(gv) : (act == 2 ? fmaxf(gv, 0.0f) : gv / (1.0f + expf(-gv)))) * uv;
     }
   }
   o.store(out + t * out_width + i);
@@ -107,7 +107,7 @@ TIE_API int tie_add_concat(int dtype, float* x, const void* delta, const float* 
 
 TIE_API int tie_glu_biased(int dtype, const void* gu, const float* bg, const float* bu, void* out, int tokens, int inter,
                            int out_width, int act, cudaStream_t s) {
-  TIE_REQUIRE(inter > 0 && out_width >= inter && (act == 0 || act == 1), "glu_biased: bad sizes inter=%d out width=%d act=%d", inter,
+  TIE_REQUIRE(inter > 0 && out_width >= inter && act >= 0 && act <= 2, "glu_biased: bad sizes inter=%d out width=%d act=%d", inter,
               out_width, act);
   const long long total = static_cast<long long>(tokens) * out_width;
   if (total <= 0) return kOk;

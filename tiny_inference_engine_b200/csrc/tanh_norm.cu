@@ -8,27 +8,9 @@
 //                   The angle is formed in double precision, so that it is the same number at position 5 and 5,000.
 #include <math.h>
 
-#include "common.cuh"
+#include "terms.cuh"
 
 namespace tie {
-
-struct Term {
-  const void* tensor;       // [T, D] in the compute type, or null
-  const float* partial;     // [splits, T, D] float, or null
-  long long stride;         // T * D
-  int splits;
-  float scale;
-};
-
-template <typename T>
-__device__ __forceinline__ float term_at(const Term& term, long long at) {
-  float v = 0.0f;
-  if (term.tensor != nullptr) v = ld(static_cast<const T*>(term.tensor) + at);
-  else if (term.partial != nullptr) {
-    for (int z = 0; z < term.splits; ++z) v += term.partial[z * term.stride + at];
-  } else return 0.0f;
-  return term.scale * v;
-}
 
 template <typename T>
 __global__ void __launch_bounds__(256) add_tanh_norm_kernel(float* __restrict__ x, Term a, Term b, const int* __restrict__ rows,
@@ -51,26 +33,6 @@ __global__ void __launch_bounds__(256) add_tanh_norm_kernel(float* __restrict__ 
 }
 
 // Four columns a thread (D a multiple of four, every pointer on a 16-byte boundary; the terms' rows likewise).
-template <typename T>
-__device__ __forceinline__ void term_add4(const Term& term, long long at, float (&v)[4]) {
-  if (term.tensor != nullptr) {
-    float d[4];
-    load4(static_cast<const T*>(term.tensor) + at, d);
-#pragma unroll
-    for (int e = 0; e < 4; ++e) v[e] = fmaf(term.scale, d[e], v[e]);
-  } else if (term.partial != nullptr) {
-    float sum[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-    for (int z = 0; z < term.splits; ++z) {
-      float d[4];
-      load4(term.partial + z * term.stride + at, d);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) sum[e] += d[e];
-    }
-#pragma unroll
-    for (int e = 0; e < 4; ++e) v[e] = fmaf(term.scale, sum[e], v[e]);
-  }
-}
-
 template <typename T>
 __global__ void __launch_bounds__(256) add_tanh_norm_vec4_kernel(float* __restrict__ x, Term a, Term b, const int* __restrict__ rows,
                                                                  float alpha, const float* __restrict__ w, const float* __restrict__ bias,

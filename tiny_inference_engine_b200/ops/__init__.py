@@ -72,8 +72,8 @@ class SplitSum:
         return out
 
 
-def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t] = float(table[ids[t]]); out is the float32 residual stream [T, D]. The table is [V, D], or the
+def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
+    """out[t] = float(table[ids[t]]) * scale; out is the float32 residual stream [T, D]. The table is [V, D], or the
     same in k-blocks, [ceil(D / 64), V, 64] (`pack_k_blocks`: what a tied output table is stored as)."""
     _dev(table, ids, out)
     T, D = out.shape
@@ -84,7 +84,7 @@ def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> None:
     _need(ids.dtype == torch.int32 and ids.numel() == T and ids.is_contiguous(), "embed: ids must be int32 [T]")
     _need(out.dtype == torch.float32 and out.is_contiguous(), "embed: output must be float32 contiguous")
     V = table.shape[1] if packed else table.shape[0]
-    call("tie_embed", dtype_code(table), table.data_ptr(), ids.data_ptr(), out.data_ptr(), T, D, V, V if packed else 0, _stream())
+    call("tie_embed", dtype_code(table), table.data_ptr(), ids.data_ptr(), out.data_ptr(), T, D, V, V if packed else 0, float(scale), _stream())
 
 
 def pack_k_blocks(w: torch.Tensor) -> torch.Tensor:
@@ -475,8 +475,9 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, partial_scratch=No
     return gemm_select.gemm(a, w, out, partial_scratch)
 
 
-def bound_gemm(w: torch.Tensor, silu: bool = False, split_many: bool = True, pack: bool = True):
+def bound_gemm(w: torch.Tensor, silu=False, split_many: bool = True, pack: bool = True):
     """A matrix product bound to one weight (gemm_select.BoundGemm): checked once, called every step.
+    `silu`: the epilogue of a gated unit, True or GATED_SILU: silu(gate) * up, GATED_RELU: max(gate, 0) * up.
     `split_many` False: above 128 tokens k is never split (the consumer wants the finished product). With `pack`
     a weight that the tensor-core kernels take is stored in k-blocks (pack_k_blocks) from here on: the product
     keeps that copy (`.w`) and the caller lets go of its own. `.rows(a, b)` is the product with rows a..b-1 of
@@ -549,6 +550,9 @@ def glu_clamped(gate_up: torch.Tensor, out: torch.Tensor, limit: float, slope: f
           "glu_clamped: gate_up must be [T, 2I] and out [T, I], same dtype, contiguous")
     call("tie_glu_clamped", dtype_code(out), gate_up.data_ptr(), out.data_ptr(), T, I, float(limit), float(slope),
          float(up_shift), _stream())
+
+
+GATED_SILU, GATED_RELU = 1, 2      # the epilogues of a gated product
 
 
 def sigmoid_gate_mul(y: torch.Tensor, gate: torch.Tensor) -> None:
@@ -962,7 +966,7 @@ def add_concat(x, delta, other, out) -> None:
          part.stride if part else 0, part.splits if part else 0, other.data_ptr(), out.data_ptr(), T, D, _stream())
 
 
-ACT_SILU, ACT_GELU_TANH = 0, 1
+ACT_SILU, ACT_GELU_TANH, ACT_RELU = 0, 1, 2
 
 
 def glu_biased(gate_up, bias_gate, bias_up, out, act: int = ACT_SILU) -> None:
@@ -984,20 +988,22 @@ ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
 
 
 def moe_route(logits, top: int, groups: int, keep: int, ids, weights, score_fn: int = ROUTE_SOFTMAX, correction=None,
-              group_top: int = 1, renorm: bool = True, weight_scale: float = 1.0) -> None:
-    """Per token: scores over all experts (`score_fn`: a softmax over the experts, or a sigmoid each); choice scores = scores +
+              group_top: int = 1, renorm: bool = True, weight_scale: float = 1.0, bias=None) -> None:
+    """Per token: scores over all experts (`score_fn`: a softmax over the experts, or a sigmoid each) of the logits plus `bias`
+    (float32 [E], optional); choice scores = scores +
     `correction` (float32 [E], optional); the `keep` best of `groups` equal blocks of consecutive experts (a group counts as the
     sum of its `group_top` largest choice scores: 1 = its best member); the `top` best experts of those by choice score. ids
     int32 [T, top], weights float32 [T, top] = the chosen experts' scores, over their sum (+ 1e-20) with `renorm`, times `weight_scale`."""
-    _dev(logits, ids, weights, correction)
+    _dev(logits, ids, weights, correction, bias)
     T, E = logits.shape
     _need(logits.dtype == torch.float32 and logits.stride(1) == 1, "moe_route: logits must be float32 rows")
     _need(ids.dtype == torch.int32 and ids.is_contiguous() and ids.shape == (T, top) and weights.dtype == torch.float32 and
           weights.is_contiguous() and weights.shape == (T, top), "moe_route: ids int32 [T, top], weights float32 [T, top]")
     _need(correction is None or (correction.dtype == torch.float32 and correction.numel() == E and correction.is_contiguous()),
           "moe_route: the correction must be float32 [experts]")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == E and bias.is_contiguous()), "moe_route: the bias must be float32 [experts]")
     call("tie_moe_route", logits.data_ptr(), logits.stride(0), T, E, top, groups, keep, int(score_fn), _ptr(correction),
-         int(group_top), int(bool(renorm)), float(weight_scale), ids.data_ptr(), weights.data_ptr(), _stream())
+         int(group_top), int(bool(renorm)), float(weight_scale), _ptr(bias), ids.data_ptr(), weights.data_ptr(), _stream())
 
 
 def moe_max_tiles(pairs: int, experts: int, block_m: int) -> int:
@@ -1313,6 +1319,9 @@ def attention_mixed_tc(q, k_cache, v_cache, out, mix, query_start, context_lens,
 
 # -- a norm without statistics and a sinusoid on the embedding (csrc/tanh_norm.cu)
 
+MAX_TERMS = 4
+
+
 class ScaledSum:
     """Sublayer outputs that join the residual stream together, each with a factor: sum_i scale_i * term_i, a term a
     tensor [T, D] in the compute dtype or a SplitSum. Norms that say `takes_scaled_sum` add the terms in float32 while
@@ -1320,8 +1329,8 @@ class ScaledSum:
 
     def __init__(self, terms):
         self.terms = [(t, float(c)) for t, c in terms if t is not None]
-        if not 1 <= len(self.terms) <= 2:
-            raise InvalidArgument(f"a scaled sum has one or two terms, got {len(self.terms)}")
+        if not 1 <= len(self.terms) <= MAX_TERMS:
+            raise InvalidArgument(f"a scaled sum has one to {MAX_TERMS} terms, got {len(self.terms)}")
 
     def materialize(self, out: torch.Tensor) -> torch.Tensor:
         acc = torch.zeros(out.shape, dtype=torch.float32, device=out.device)      # off the product path: toy parts and tests only
@@ -1338,6 +1347,7 @@ def add_tanh_norm(x: torch.Tensor, delta, alpha: float, weight: torch.Tensor, bi
     out's dtype, a SplitSum, or a ScaledSum of up to two of those. With `rows` (int32 [R]) out[i] comes from row rows[i]
     and x is left as it is."""
     terms = delta.terms if isinstance(delta, ScaledSum) else ([(delta, 1.0)] if delta is not None else [])
+    _need(len(terms) <= 2, "add_tanh_norm: at most two terms")
     _dev(x, weight, bias, out, rows)
     D, n = x.shape[-1], out.shape[0]
     _need(x.dtype == torch.float32 and x.is_contiguous(), "add_tanh_norm: x must be float32 contiguous")
@@ -1553,3 +1563,218 @@ def time_mix_out(o, gate, weight, eps: float, out, heads: int, dim: int, h, stat
     call("tie_time_mix_out", dtype_code(out), o.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), float(eps), out.data_ptr(), T,
          heads, dim, h.data_ptr(), D, state.data_ptr(), state.stride(0), prev_off, ctx.seq_of_row.data_ptr(), ctx.query_start.data_ptr(),
          ctx.state_slots.data_ptr(), _stream())
+
+
+# -- a norm with mean and variance, sums into the stream (csrc/layer_norm.cu)
+
+def flat_terms(delta) -> list:
+    """(tensor or SplitSum, factor) pairs of what is still to join the residual stream: a tensor, a SplitSum, a ScaledSum or None."""
+    if delta is None:
+        return []
+    return list(delta.terms) if isinstance(delta, ScaledSum) else [(delta, 1.0)]
+
+
+def _term_args(delta, x, dtype, what: str) -> list:
+    terms, args = flat_terms(delta), []
+    for t, c in terms + [(None, 0.0)] * (MAX_TERMS - len(terms)):
+        if isinstance(t, SplitSum):
+            _need(t.M == x.shape[0] and t.N == x.shape[1], f"{what}: partial sums do not match x")
+            args += [0, t.partial.data_ptr(), t.stride, t.splits, c]
+        else:
+            if t is not None:
+                _dev(t)
+                _need(t.dtype == dtype and t.shape == x.shape and t.is_contiguous(), f"{what}: a term must have x's shape and the compute dtype")
+            args += [_ptr(t), 0, 0, 0, c]
+    return args
+
+
+def add_layer_norm(x, delta, weight, bias, eps: float, out, rows=None) -> None:
+    """x += delta (when given; float32, in place), out = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias in out's
+    dtype. `delta`: a tensor in out's dtype, a SplitSum, or a ScaledSum of up to four of those. With `rows` (int32 [R]) out[i]
+    comes from row rows[i] and x is left as it is."""
+    _dev(x, weight, bias, out, rows)
+    D, n = x.shape[-1], out.shape[0]
+    _need(x.dtype == torch.float32 and x.is_contiguous(), "add_layer_norm: x must be float32 contiguous")
+    _need(all(w.dtype == torch.float32 and w.numel() == D for w in (weight, bias)), "add_layer_norm: weight and bias must be float32 [D]")
+    _need(out.shape[-1] == D and out.is_contiguous(), "add_layer_norm: out must be [n, D] contiguous")
+    _need(rows is None and n == x.shape[0] or rows is not None and rows.dtype == torch.int32 and rows.numel() == n,
+          "add_layer_norm: out must have x's rows, or rows must be int32 [n]")
+    call("tie_add_layer_norm", dtype_code(out), x.data_ptr(), *_term_args(delta, x, out.dtype, "add_layer_norm"), _ptr(rows),
+         weight.data_ptr(), bias.data_ptr(), float(eps), out.data_ptr(), n, D, _stream())
+
+
+def stream_add(x, delta, dtype, other=None, vec=None) -> None:
+    """x += delta (as for `add_layer_norm`; tensors of `dtype`), then += other (float32 rows), then += vec (float32 [D], every row)."""
+    _dev(x, other, vec)
+    T, D = x.shape
+    _need(x.dtype == torch.float32 and x.is_contiguous(), "stream_add: x must be float32 contiguous")
+    _need(other is None or (other.dtype == torch.float32 and other.is_contiguous() and other.shape == x.shape), "stream_add: other must be float32 rows of x's shape")
+    _need(vec is None or (vec.dtype == torch.float32 and vec.is_contiguous() and vec.numel() == D), "stream_add: vec must be float32 [D]")
+    call("tie_stream_add", _DT[dtype], x.data_ptr(), *_term_args(delta, x, dtype, "stream_add"), _ptr(other), _ptr(vec), T, D, _stream())
+
+
+def cap_rows(x, cap: float) -> None:
+    """x = cap * tanh(x / cap) for float32 rows, in place."""
+    _dev(x)
+    _need(x.dim() == 2 and x.dtype == torch.float32 and x.stride(1) == 1, "cap_rows: x must be float32 rows")
+    call("tie_cap_rows", x.data_ptr(), x.stride(0), x.shape[0], x.shape[1], float(cap), _stream())
+
+
+# -- short causal convolutions over time (csrc/short_conv.cu)
+
+def conv_tile(ctx) -> int:
+    """Rows a thread of the convolution kernels walks down: one where every sequence brings one token. (Where a step is cut
+    into tiles decides which kernel moves a sequence's last inputs into its slot, nothing else.)"""
+    return 1 if ctx.multi_seqs == 0 else 8
+
+
+def _conv_args(proj, col0, channels, taps, w, pre, post, state, tail_off, what):
+    _dev(proj, w, pre, post, state)
+    _need(proj.dim() == 2 and proj.stride(1) == 1 and col0 + channels <= proj.shape[1], f"{what}: channels outside the projection")
+    _need(w.dtype == torch.float32 and w.is_contiguous() and w.shape == (taps, channels), f"{what}: weights must be float32 [taps, channels]")
+    for b in (pre, post):
+        _need(b is None or (b.dtype == torch.float32 and b.numel() == channels and b.is_contiguous()), f"{what}: a bias must be float32 [channels]")
+    if taps > 1:
+        _need(state is not None and state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1 and
+              tail_off + (taps - 1) * channels <= state.shape[1], f"{what}: state rows too short")
+
+
+def short_conv_act(proj, col0: int, w, post, state, tail_off: int, ctx, out, silu: bool = True) -> None:
+    """out[t, c] = act(post[c] + sum_j w[j, c] u_(t - taps + 1 + j)[c]), u the columns col0.. of `proj` (w float32 [taps, channels],
+    the last row weighs the current token), zeros ahead of a sequence. The last taps - 1 inputs of every sequence sit in its row
+    of `state` from tail_off on ([taps - 1, channels] float32, oldest first) and are moved on. out in proj's dtype."""
+    taps, channels = w.shape
+    _conv_args(proj, col0, channels, taps, w, None, post, state, tail_off, "short_conv_act")
+    T, tile = proj.shape[0], conv_tile(ctx)
+    _need(out.dtype == proj.dtype and out.shape == (T, channels) and out.stride(1) == 1, "short_conv_act: out must be [T, channels] in proj's dtype")
+    st = (_ptr(state), state.stride(0)) if taps > 1 else (0, 0)
+    call("tie_short_conv_act", dtype_code(proj), proj.data_ptr(), proj.stride(0), col0, channels, taps, T, tile, w.data_ptr(), 0, _ptr(post),
+         *st, tail_off, ctx.seq_of_row.data_ptr(), ctx.query_start.data_ptr(), ctx.state_slots.data_ptr(), 1 if silu else 0, out.data_ptr(),
+         out.stride(0), _stream())
+    _conv_tail(proj, col0, channels, taps, tile, None, state, tail_off, ctx)
+
+
+def _conv_tail(proj, col0, channels, taps, tile, pre, state, tail_off, ctx) -> None:
+    if ctx.multi_seqs > 0 and taps > 1:
+        call("tie_conv_tail", dtype_code(proj), proj.data_ptr(), proj.stride(0), col0, channels, taps, tile, _ptr(pre), state.data_ptr(),
+             state.stride(0), tail_off, ctx.query_start.data_ptr(), ctx.state_slots.data_ptr(), ctx.multi_seqs, _stream())
+
+
+def conv_rope_append(proj, col0: int, k_col: int, w, pre, state, tail_off: int, ctx, turns, slots, k_cache, v_cache, q_out, q_heads: int,
+                     kv_heads: int, dim: int) -> None:
+    """The q heads (channels 0.. behind column col0) and the k heads (channels k_col..) of `proj` plus `pre` (a bias, float32
+    [channels]) through a causal convolution per channel (as `short_conv_act`, no activation). What a k head becomes is its
+    value (value plane); with the first 2 * len(turns) dimensions of each head turned in neighbouring pairs by
+    position * turns[i] turns (float64) it is its key (key plane), and likewise q into q_out [T, q_heads * dim]."""
+    taps, channels = w.shape
+    _conv_args(proj, col0, channels, taps, w, pre, None, state, tail_off, "conv_rope_append")
+    T, tile = proj.shape[0], conv_tile(ctx)
+    _check_kv_planes(k_cache, v_cache, kv_heads, dim, dim)
+    _dev(turns, slots, k_cache, v_cache, q_out)
+    _need(k_cache.dtype == proj.dtype and q_out.dtype == proj.dtype and q_out.is_contiguous() and q_out.shape == (T, q_heads * dim),
+          "conv_rope_append: q_out must be [T, q_heads * dim] in proj's dtype, the planes too")
+    _need(turns is None or turns.dtype == torch.float64, "conv_rope_append: turns must be float64")
+    _need(slots.dtype == torch.int32 and slots.numel() == T and ctx.positions.numel() == T, "conv_rope_append: slots must be int32 [T]")
+    st = (_ptr(state), state.stride(0)) if taps > 1 else (0, 0)
+    call("tie_conv_rope_append", dtype_code(proj), proj.data_ptr(), proj.stride(0), col0, channels, taps, T, tile, w.data_ptr(), _ptr(pre), *st,
+         tail_off, ctx.seq_of_row.data_ptr(), ctx.query_start.data_ptr(), ctx.state_slots.data_ptr(), ctx.positions.data_ptr(), _ptr(turns),
+         2 * turns.numel() if turns is not None else 0, slots.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), q_out.data_ptr(), q_heads,
+         kv_heads, dim, k_cache.shape[2], k_col, _stream())
+    _conv_tail(proj, col0, channels, taps, tile, pre, state, tail_off, ctx)
+
+
+# -- a diagonal recurrence with a step size per token and channel (csrc/selective_scan.cu)
+
+def selective_scan(x, z, low, b_off: int, c_off: int, raw, bias, a2, skip, state, ctx, out) -> None:
+    """dt = softplus(raw + bias); S <- exp2(dt a2) S + dt x B; y = S C + skip x; out = y silu(z), over each sequence's rows of the
+    step. x, z [T, inner], `low` (B at column b_off, C at c_off) and out in the compute dtype; raw float32 [T, inner]; bias, skip
+    float32 [inner]; a2 float32 [inner, states] (A times log2 e). S [inner, states] sits at the start of the sequence's row of `state`."""
+    _dev(x, z, low, raw, bias, a2, skip, state, out)
+    T, inner = x.shape
+    states = a2.shape[1]
+    for t in (x, z):
+        _need(t.shape == (T, inner) and t.stride(1) == 1 and t.dtype == out.dtype, "selective_scan: x and z must be [T, inner] in out's dtype")
+    _need(low.dim() == 2 and low.stride(1) == 1 and low.dtype == out.dtype and low.shape[0] == T and low.shape[1] >= c_off + states,
+          "selective_scan: B and C outside their rows")
+    _need(raw.dtype == torch.float32 and raw.is_contiguous() and raw.shape == (T, inner), "selective_scan: raw must be float32 [T, inner]")
+    _need(a2.dtype == torch.float32 and a2.is_contiguous() and a2.shape[0] == inner and
+          all(v.dtype == torch.float32 and v.numel() == inner for v in (bias, skip)), "selective_scan: bias, skip float32 [inner], a2 float32 [inner, states]")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1 and state.shape[1] >= inner * states, "selective_scan: state rows too short")
+    _need(out.is_contiguous() and out.shape == (T, inner), "selective_scan: out must be [T, inner] contiguous")
+    call("tie_selective_scan", dtype_code(out), x.data_ptr(), x.stride(0), z.data_ptr(), z.stride(0), low.data_ptr(), low.stride(0), b_off, c_off,
+         raw.data_ptr(), bias.data_ptr(), a2.data_ptr(), skip.data_ptr(), state.data_ptr(), state.stride(0), ctx.query_start.data_ptr(),
+         ctx.state_slots.data_ptr(), ctx.S, inner, states, out.data_ptr(), 1 if ctx.multi_seqs > 0 else 0, _stream())
+
+
+def act_split(proj, q_off: int, k_off: int, v_off: int, qn, kn, vn, silu: bool = True) -> None:
+    """The q, k and v columns of `proj` behind the SiLU (or as they are) as float32 rows qn, kn [T, nqk], vn [T, nv]."""
+    _dev(proj, qn, kn, vn)
+    T, nqk, nv = proj.shape[0], qn.shape[1], vn.shape[1]
+    _need(proj.dim() == 2 and proj.stride(1) == 1 and max(q_off + nqk, k_off + nqk, v_off + nv) <= proj.shape[1], "act_split: columns outside the projection")
+    for t, n in ((qn, nqk), (kn, nqk), (vn, nv)):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n), "act_split: outputs must be float32 [T, n]")
+    call("tie_act_split", dtype_code(proj), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, T, nqk, nv, 1 if silu else 0, qn.data_ptr(),
+         kn.data_ptr(), vn.data_ptr(), _stream())
+
+
+# -- attention in a window beside which the first keys stay visible, with capped scores and a sink per head
+
+def _kept_sink(sink, q_heads):
+    _dev(sink)
+    _need(sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == q_heads), "attention: sinks must be float32 [q_heads]")
+    return _ptr(sink)
+
+
+def attention_kept_rows(q, k_cache, v_cache, out, seq_of_row, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim,
+                        scale: float, window: int = 0, keep_first: int = 0, softcap: float = 0.0, sink=None) -> None:
+    """`attention_rows_dv` in which position i sees j <= i with i - j < window or j < keep_first, score <- softcap tanh(score / softcap)
+    (softcap > 0), and exp(sink[h]) is one more term of head h's softmax denominator (sink float32 [q_heads] or None)."""
+    _dev(q, k_cache, v_cache, out, seq_of_row, query_start, context_lens, block_tables)
+    S = _attn_common_dv(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim)
+    _need(seq_of_row.dtype == torch.int32 and seq_of_row.numel() == q.shape[0], "attention: seq_of_row must be int32 [T]")
+    call("tie_attention_kept_rows", dtype_code(q), q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
+         seq_of_row.data_ptr(), query_start.data_ptr(), context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], q.shape[0], S,
+         q_heads, kv_heads, head_dim, v_dim, k_cache.shape[2], int(window), int(keep_first), float(scale), float(softcap),
+         _kept_sink(sink, q_heads), _stream())
+
+
+def attention_kept_split(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim, scale: float,
+                         seq_list, n_list: int, split_keys: int, max_splits: int, scratch, window: int = 0, keep_first: int = 0,
+                         softcap: float = 0.0, sink=None) -> None:
+    """The same for sequences that bring one token each, the keys they see in splits of `split_keys`; scratch as for `attention_split_dv`."""
+    _dev(q, k_cache, v_cache, out, query_start, context_lens, block_tables, seq_list, scratch)
+    S = _attn_common_dv(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim)
+    _need(seq_list.dtype == torch.int32 and seq_list.numel() >= n_list, "attention: seq_list must be int32 [n_list]")
+    _need(scratch.dtype == torch.float32 and
+          scratch.numel() >= attention_split_scratch_floats(n_list, q_heads, v_dim, max_splits), "attention: scratch too small")
+    call("tie_attention_kept_split", dtype_code(q), q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
+         query_start.data_ptr(), context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], S, q_heads, kv_heads, head_dim, v_dim,
+         k_cache.shape[2], int(window), int(keep_first), float(scale), float(softcap), _kept_sink(sink, q_heads), seq_list.data_ptr(), n_list,
+         split_keys, max_splits, scratch.data_ptr(), _stream())
+
+
+def attention_prompt_kept(q, k_cache, v_cache, out, query_start, context_lens, block_tables, n_seqs: int, max_queries: int, q_heads, kv_heads,
+                          head_dim, scale: float, window: int = 0, keep_first: int = 0, softcap: float = 0.0, sink=None) -> None:
+    """`attention_prompt_tma` (exact weights) with the options of `attention_kept_rows`."""
+    _dev(q, k_cache, v_cache, out, query_start, context_lens, block_tables)
+    _attn_common(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim)
+    call("tie_attention_prompt_kept", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), query_start.data_ptr(),
+         context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], n_seqs, max_queries, q_heads, kv_heads, head_dim,
+         k_cache.shape[2], k_cache.shape[0], int(window), int(keep_first), float(scale), float(softcap), _kept_sink(sink, q_heads), _stream())
+
+
+def attention_decode_kept(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, scale: float,
+                          first: int, n_list: int, split_keys: int, max_splits: int, scratch, counters, window: int = 0, keep_first: int = 0,
+                          softcap: float = 0.0, sink=None, cluster: bool = False) -> None:
+    """`attention_decode_tma` (exact weights, sequences first .. first + n_list - 1) with the options of `attention_kept_rows`. The
+    kept keys come on top of the first split's own."""
+    _dev(q, k_cache, v_cache, out, query_start, context_lens, block_tables, scratch, counters)
+    S = _attn_common(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim)
+    _need(0 <= first and first + n_list <= S, "attention: sequences outside the step")
+    _need(scratch.dtype == torch.float32 and
+          scratch.numel() >= attention_split_scratch_floats(n_list, q_heads, head_dim, max_splits), "attention: scratch too small")
+    _need(counters.dtype == torch.int32 and counters.numel() >= n_list * kv_heads, "attention: counters too small")
+    call("tie_attention_decode_kept", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), query_start.data_ptr(),
+         context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], q_heads, kv_heads, head_dim, k_cache.shape[2],
+         k_cache.shape[0], int(window), int(keep_first), float(scale), float(softcap), _kept_sink(sink, q_heads), 0, first, n_list, split_keys,
+         max_splits, scratch.data_ptr(), counters.data_ptr(), 1 if cluster else 0, _stream())

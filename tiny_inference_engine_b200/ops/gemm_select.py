@@ -157,7 +157,7 @@ def pair_width(M: int, N: int, K: int, pairs: int) -> int:
 
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, transposed=None, bn=None, splits=None, scratch=None,
-            silu: bool = False, partial_scratch=None, deep=None, pair=None, checked: bool = False):
+            silu=False, partial_scratch=None, deep=None, pair=None, checked: bool = False):
     """The tensor-core product; the tiling can be forced (tests). Returns `out`, or a SplitSum when
     `partial_scratch` is given and k is split."""
     global _ops
@@ -176,7 +176,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, transposed=None
         pair = transposed is None and bn is None and splits is None and pair_takes(M, N)
     if pair:
         _call("tie_gemm_tc2", dtype_code(out), a.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, a.stride(0),
-              w.stride(0), out.stride(0), 1 if silu else 0, 0, 0, bn if bn in PAIR_WIDTHS else pair_width(M, N, K, resident_pairs()),
+              w.stride(0), out.stride(0), int(silu), 0, 0, bn if bn in PAIR_WIDTHS else pair_width(M, N, K, resident_pairs()),
               _stream())
         return out
     t, b, s = plan(M, N, K)
@@ -193,7 +193,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, transposed=None
     elif splits > 1 and scratch is None:
         scratch = _scratch_for(splits * M * N, a.device)
     _call("tie_gemm_tc", dtype_code(out), a.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, a.stride(0),
-          w.stride(0), out.stride(0), transposed, bn, splits, scratch.data_ptr() if splits > 1 else 0, 1 if silu else 0,
+          w.stride(0), out.stride(0), transposed, bn, splits, scratch.data_ptr() if splits > 1 else 0, int(silu),
           0 if leave else 1, int(deep if deep is not None else (not transposed or bn >= 128)), 0, 0, _stream())
     if leave:
         return SplitSum(scratch, _library().tie_gemm_tc_real_splits(K, splits), M, N)
@@ -224,12 +224,12 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, partial_scratch=No
     return out
 
 
-def gemm_silu(a: torch.Tensor, w_blocks: torch.Tensor, out: torch.Tensor) -> None:
+def gemm_silu(a: torch.Tensor, w_blocks: torch.Tensor, out: torch.Tensor, act: int = 1) -> None:
     from . import _need
     _need(w_blocks.shape[0] % 32 == 0 and tc_takes(a, w_blocks, out),
           "gemm_silu: needs bfloat16 operands TMA can address and gate/up rows in blocks of 16")
     if a.shape[0] > 0:
-        gemm_tc(a, w_blocks, out, silu=True)
+        gemm_tc(a, w_blocks, out, silu=act)
 
 
 class BoundGemm:
@@ -244,8 +244,8 @@ class BoundGemm:
     [ceil(K / 64), rows, 64] and `packed_rows` its number of rows; `.rows(a, b)` gives the product with a slice of
     its rows (the q rows of a stacked q/k/v weight) over the same memory."""
 
-    def __init__(self, w: torch.Tensor, silu: bool = False, split_many: bool = True, pack: bool = True, _slice=None):
-        self.silu, self.split_many = silu, split_many
+    def __init__(self, w: torch.Tensor, silu=False, split_many: bool = True, pack: bool = True, _slice=None):
+        self.silu, self.split_many = int(silu), split_many      # 0: none, 1: the SiLU, 2: the ReLU of a gated unit
         if _slice is not None:              # rows [row0, row0 + N) of a packed weight
             parent, row0, n = _slice
             self.w, self.N, self.K, self.packed_rows, self.row0, self.fast = parent.w, n, parent.K, parent.packed_rows, row0, True
@@ -300,7 +300,7 @@ class BoundGemm:
                 and out.shape[0] == M and out.dtype in (torch.bfloat16, torch.float32)):
             w = self.row_major()
             if self.silu:
-                gemm_silu(a, w, out)
+                gemm_silu(a, w, out, self.silu)
                 return out
             return gemm(a, w, out, partial_scratch)
         global _ops
@@ -312,7 +312,7 @@ class BoundGemm:
         code = 1 if out.dtype == torch.bfloat16 else 0
         if pair:
             _call("tie_gemm_tc2", code, a.data_ptr(), self.w_ptr, out.data_ptr(), M, self.N, self.K, a.stride(0), self.ldw,
-                  out.stride(0), 1 if self.silu else 0, self.packed_rows, self.row0, bn, _stream())
+                  out.stride(0), self.silu, self.packed_rows, self.row0, bn, _stream())
             return out
         leave = splits > 1 and partial_scratch is not None
         scratch = 0
@@ -323,7 +323,7 @@ class BoundGemm:
             buf = _scratch_for(splits * M * self.N, a.device)
             scratch = buf.data_ptr()
         _call("tie_gemm_tc", code, a.data_ptr(), self.w_ptr, out.data_ptr(), M, self.N, self.K, a.stride(0), self.ldw, out.stride(0),
-              t, bn, splits, scratch, 1 if self.silu else 0, 0 if leave else 1, deep, self.packed_rows, self.row0, _stream())
+              t, bn, splits, scratch, self.silu, 0 if leave else 1, deep, self.packed_rows, self.row0, _stream())
         if leave:
             return SplitSum(buf, real, M, self.N)
         return out

@@ -14,9 +14,10 @@ _LOCK = threading.Lock()
 _LIB = None
 
 P, I, L, F = c_void_p, c_int, c_longlong, c_float
+_TERMS = [P, P, L, I, F] * 4      # sums into the residual stream: (tensor, partial sums, stride, splits, factor) each
 
 _SIGNATURES = {
-    "tie_embed": [I, P, P, P, I, I, I, I, P],
+    "tie_embed": [I, P, P, P, I, I, I, I, F, P],
     "tie_scatter_ids": [P, P, P, P, I, P],
     "tie_add_rmsnorm": [I, P, P, P, L, I, P, P, F, P, I, I, P],
     "tie_rmsnorm_rows": [I, P, L, P, F, P, L, I, L, P],
@@ -62,7 +63,7 @@ _SIGNATURES = {
     "tie_attention_latent_split": [P, L, P, P, P, P, I, I, I, I, I, I, F, P, I, I, I, P, P],
     "tie_add_concat": [I, P, P, P, L, I, P, P, I, I, P],
     "tie_glu_biased": [I, P, P, P, P, I, I, I, I, P],
-    "tie_moe_route": [P, L, I, I, I, I, I, I, P, I, I, F, P, P, P],
+    "tie_moe_route": [P, L, I, I, I, I, I, I, P, I, I, F, P, P, P, P],
     "tie_moe_align": [P, I, I, I, P, P, P, P],
     "tie_moe_gemm": [I, I, I, P, L, P, L, P, L, P, L, P, P, P, P, I, I, I, I, I, P],
     "tie_moe_gather": [I, P, L, P, P, I, I, P, I, I, P],
@@ -91,6 +92,18 @@ _SIGNATURES = {
     "tie_time_mix_prep": [I, P, L, I, I, I, I, I, P, P, P, P, P, P, I, I, P],
     "tie_time_mix_out": [I, P, P, L, P, F, P, I, I, I, P, I, P, L, L, P, P, P, P],
     "tie_two_branch_unit": [I, P, P, L, F, F, P],
+    "tie_add_layer_norm": [I, P, *_TERMS, P, P, P, F, P, I, I, P],
+    "tie_stream_add": [I, P, *_TERMS, P, P, I, I, P],
+    "tie_cap_rows": [P, L, I, I, F, P],
+    "tie_short_conv_act": [I, P, L, I, I, I, I, I, P, P, P, P, L, L, P, P, P, I, P, L, P],
+    "tie_conv_rope_append": [I, P, L, I, I, I, I, I, P, P, P, L, L, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, P],
+    "tie_conv_tail": [I, P, L, I, I, I, I, P, P, L, L, P, P, I, P],
+    "tie_selective_scan": [I, P, L, P, L, P, L, I, I, P, P, P, P, P, L, P, P, I, I, I, P, I, P],
+    "tie_act_split": [I, P, L, I, I, I, I, I, I, I, P, P, P, P],
+    "tie_attention_kept_rows": [I, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, P, P],
+    "tie_attention_kept_split": [I, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, P, P, I, I, I, P, P],
+    "tie_attention_prompt_kept": [P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, P, P],
+    "tie_attention_decode_kept": [P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P, P, I, I, I, I, P, P, I, P],
     "tie_attention_mixed": [I, P, L, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P, I, I, I, P, P],
 }
 

@@ -4,7 +4,7 @@ from .base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSI
                    register_part, to_compute)
 from . import (norm, position, attention, gated_attention, delta, feed_forward, block, embedding,  # noqa: F401  (register the built-in kinds)
                latent_attention, linear_attention, state_space, experts, stream_input, head_mix_attention,
-               score_map_attention, time_mix)
+               score_map_attention, time_mix, conv_attention, selective_scan)
 from .attention import GQAttention
 from .block import PreNormBlock
 from .embedding import LMHead, TokenEmbedding

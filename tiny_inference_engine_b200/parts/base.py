@@ -23,12 +23,14 @@ class CacheNeed:
     """What a mixer wants of the paged cache: keys and values of `kv_heads` x `head_dim` per
     token; kind "full" keeps every token, "window" only the last `window`. `value_dim` is the
     size of a value head where it differs from a key head's (0: the same; -1: the cache keeps keys only and
-    the mixer finds a token's value inside its key, as attention over one latent per token does)."""
+    the mixer finds a token's value inside its key, as attention over one latent per token does). `keep_first`: a
+    "window" also keeps that many of the sequence's first tokens, at their own places."""
     kind: str
     kv_heads: int
     head_dim: int
     window: int = 0
     value_dim: int = 0
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

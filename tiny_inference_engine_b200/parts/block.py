@@ -249,6 +249,42 @@ class ParallelBlock(Block):
         return None
 
 
+class SharedNormBlock(Block):
+    """One norm, and both sublayers side by side on its output: h = norm(x), x += mixer(h) + ffn(h). A layer may have no
+    feed-forward. The block adds nothing itself: it hands on the sublayers' outputs (tensors, partial sums of split products,
+    sums with factors) as one `ops.ScaledSum`, which the next layer's norm adds in float32 while it reads the stream. The two
+    sublayers' outputs must lie in buffers of their own."""
+    launches_only = False
+
+    def __init__(self, layer_spec, dtype, prefix: str = ""):
+        self.norm = build_part("norm", layer_spec.mixer_norm, dtype)
+        self.mixer = build_part("mixer", layer_spec.mixer, dtype)
+        self.has_ffn = layer_spec.ffn is not None
+        self.ffn = build_part("feed_forward", layer_spec.ffn, dtype) if self.has_ffn else None
+        self.dtype = dtype
+        self.parts = (self.norm, self.mixer) + ((self.ffn,) if self.has_ffn else ())
+
+    def needs(self):
+        n = {}
+        for p in self.parts:
+            n.update(p.needs())
+        return n
+
+    def bind(self, get):
+        for p in self.parts:
+            p.bind(get)
+
+    def forward(self, x, pending, ctx, cache, state):
+        from .. import ops
+        h = ctx.ws.rows("block.normed", x.shape[0], x.shape[1], self.dtype)
+        self.norm.add_norm(x, as_delta(pending, self.norm, ctx, "block.delta"), h)
+        mixed = self.mixer.forward(h, ctx, cache, state)
+        if not self.has_ffn:
+            return mixed
+        return ops.ScaledSum(ops.flat_terms(mixed) + ops.flat_terms(self.ffn.forward(h, ctx)))
+
+
 register_part("block", "prenorm", PreNormBlock, replace=True)
+register_part("block", "shared_norm", SharedNormBlock, replace=True)
 register_part("block", "sandwich_norm", SandwichNormBlock, replace=True)
 register_part("block", "parallel", ParallelBlock, replace=True)

@@ -11,9 +11,12 @@ from .base import Embedding, OutputHead, register_part, to_compute
 
 
 class TokenEmbedding(Embedding):
+    """x[t] = table[id] * scale, the product in float32 (`scale` 1 when absent)."""
+
     def __init__(self, spec, dtype, prefix: str = ""):
         self.name = spec["name"]
         self.vocab, self.hidden = int(spec["vocab_size"]), int(spec["hidden_size"])
+        self.scale = float(spec.params.get("scale", 1.0))
         self.dtype = dtype
         self.table = None
 
@@ -27,7 +30,7 @@ class TokenEmbedding(Embedding):
         self.table = self.product.w
 
     def forward(self, tokens, x):
-        ops.embed(self.table, tokens, x)
+        ops.embed(self.table, tokens, x, self.scale)
 
 
 class NormedTokenEmbedding(TokenEmbedding):
@@ -110,6 +113,7 @@ class LMHead(OutputHead):
         self.tied = bool(spec["tied"])
         self.vocab, self.hidden = int(spec["vocab_size"]), int(spec["hidden_size"])
         self.logit_scale = float(spec.params.get("logit_scale", 1.0))      # a constant factor on the float32 logits
+        self.softcap = float(spec.params.get("softcap") or 0.0)            # > 0: logits <- softcap * tanh(logits / softcap), float32
         self.dtype = dtype
         self.embedding = embedding
         self.weight = None
@@ -131,6 +135,8 @@ class LMHead(OutputHead):
         self.product(last, logits)
         if self.logit_scale != 1.0:
             ops.scale_rows(logits, self.logit_scale)
+        if self.softcap > 0.0:
+            ops.cap_rows(logits, self.softcap)
 
 
 register_part("embedding", "token_embedding", TokenEmbedding, replace=True)

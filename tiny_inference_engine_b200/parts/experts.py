@@ -1,11 +1,12 @@
 """A feed-forward of many small experts of which each token uses a few.
 
-    s      = softmax(h Wr^T) over all experts, or sigmoid(h Wr^T) each (`score`: "softmax" | "sigmoid")   float32
+    z      = h Wr^T, plus a bias per expert                         (`router_bias`: a tensor `<prefix>router.b` [experts])   float32
+    s      = softmax(z) over all experts, or sigmoid(z) each (`score`: "softmax" | "sigmoid")   float32
     c      = s + correction                                         (`correction`: a tensor `<prefix>correction` [experts]; else c = s)
     chosen = the `top` experts with the largest c among the experts of the `group_keep` best of `group_count` equal
              blocks of consecutive experts (a block's score is the sum of its `group_top` largest c, 1: its best
              member's; ties go to the lower index; experts of other blocks count as minus infinity)
-    weight = s[chosen] / (sum of s[chosen] + 1e-20), or s[chosen] as it is (`renorm` false), times `weight_scale`
+    weight = s[chosen] / (sum of s[chosen] + 1e-20) (with softmax scores: the softmax over the chosen logits alone), or s[chosen] as it is (`renorm` false), times `weight_scale`
     out    = sum over chosen of weight * expert(h)
     expert = down(g * sigmoid(slope * g) * (u + up_shift)),  g = min(gate(h), limit), u = clamp(up(h), -limit, limit)
              (`limit` None: no clamps; with slope 1 and up_shift 0 that is silu(gate(h)) * up(h))
@@ -16,7 +17,7 @@ and two grouped products run over that list, the clamped unit between them. The 
 weight * result as float32 partial sums [top, tokens, hidden], which the block's next residual add sums in order:
 the weighted sum over experts happens in float32 in the residual add itself. What a token computes depends on its
 own experts only, never on what else is in the step. params: `hidden_size`, `intermediate_size`, `num_experts`, `top`,
-`group_count`, `group_keep`, `group_top`, `score`, `correction`, `renorm`, `weight_scale`, `limit`, `slope`, `up_shift`; tensors `<prefix>router` and `<prefix>e<i>.gate|up|down`.
+`group_count`, `group_keep`, `group_top`, `score`, `router_bias`, `correction`, `renorm`, `weight_scale`, `limit`, `slope`, `up_shift`; tensors `<prefix>router` and `<prefix>e<i>.gate|up|down`.
 """
 from __future__ import annotations
 
@@ -50,6 +51,8 @@ class RoutedExperts(FeedForward):
         self.group_top, self.renorm = int(p.get("group_top", 1)), bool(p.get("renorm", True))
         self.has_correction = bool(p.get("correction", False))
         self.correction = None
+        self.has_router_bias = bool(p.get("router_bias", False))
+        self.router_bias = None
         E, G = self.experts, self.group_count
         if min(E, self.top, G, self.group_keep, self.inter) <= 0 or E % G or self.group_keep > G or \
                 self.top > self.group_keep * (E // G) or self.top > 32:
@@ -64,6 +67,8 @@ class RoutedExperts(FeedForward):
         n = {self.prefix + "router": TensorNeed((self.experts, self.hidden))}
         if self.has_correction:
             n[self.prefix + "correction"] = TensorNeed((self.experts,))
+        if self.has_router_bias:
+            n[self.prefix + "router.b"] = TensorNeed((self.experts,), "norm")
         for e in range(self.experts):
             n[self._expert(e, "gate")] = TensorNeed((self.inter, self.hidden))
             n[self._expert(e, "up")] = TensorNeed((self.inter, self.hidden))
@@ -81,6 +86,8 @@ class RoutedExperts(FeedForward):
         self.router_rows = rows
         if self.has_correction:
             self.correction = get(self.prefix + "correction").to(torch.float32).contiguous()
+        if self.has_router_bias:
+            self.router_bias = get(self.prefix + "router.b").to(torch.float32).contiguous()
         # [experts, 2 * inter, hidden]: an expert's gate rows, then its up rows; [experts, hidden, inter]
         w_gate_up = torch.stack([torch.cat([to_compute(get(self._expert(e, "gate")), self.dtype),
                                             to_compute(get(self._expert(e, "up")), self.dtype)], dim=0) for e in range(E)]).contiguous()
@@ -103,7 +110,8 @@ class RoutedExperts(FeedForward):
         ids = ctx.ws.rows("moe.ids", T, top, torch.int32)
         weights = ctx.ws.rows("moe.weights", T, top, torch.float32)
         ops.moe_route(logits[:, :E], top, self.group_count, self.group_keep, ids, weights, score_fn=self.score_fn,
-                      correction=self.correction, group_top=self.group_top, renorm=self.renorm, weight_scale=self.weight_scale)
+                      correction=self.correction, group_top=self.group_top, renorm=self.renorm, weight_scale=self.weight_scale,
+                      bias=self.router_bias)
         pairs = T * top
         few = pairs <= 8 * E      # an expert has a few rows: a warp per output column streams its weights once
         if self.in_blocks:

@@ -1,4 +1,4 @@
-"""SwiGLU feed-forward: down(silu(gate(h)) * up(h)), silu(g) = g / (1 + exp(-g))
+"""Gated feed-forwards. SwiGLU: down(silu(gate(h)) * up(h)), silu(g) = g / (1 + exp(-g))
 (src/model/qwen3.cpp:235-238, src/backend/cpu/cpu_backend.cpp:195-207). Gate and up are
 stacked into one weight so that one product reads h once."""
 from __future__ import annotations
@@ -11,31 +11,38 @@ from .base import FeedForward, register_part, to_compute
 
 
 class SwiGLU(FeedForward):
+    """down(act(gate(h)) * up(h)), act the SiLU or, with `activation` "relu", max(g, 0). params: `hidden_size`,
+    `intermediate_size`, `activation`, and the three tensors' names (`gate`, `up`, `down`) after `prefix`."""
     launches_only = True
+    EPILOGUES = {"silu": ops.GATED_SILU, "relu": ops.GATED_RELU}
 
     def __init__(self, spec, dtype, prefix: str = ""):
         p = spec.params
         self.prefix = prefix + p.get("prefix", "")
         self.hidden = int(p["hidden_size"])
         self.inter = int(p["intermediate_size"])
+        act = p.get("activation", "silu")
+        if act not in self.EPILOGUES:
+            from ..errors import UnsupportedError
+            raise UnsupportedError(f"no activation '{act}' (known: {', '.join(sorted(self.EPILOGUES))})")
+        self.epilogue = self.EPILOGUES[act]
+        self.names = tuple(self.prefix + p.get(k, k + "_proj.weight") for k in ("gate", "up", "down"))
         self.dtype = dtype
         self.w_gate_up = self.w_down = None
 
     def needs(self):
-        return {self.prefix + "gate_proj.weight": TensorNeed((self.inter, self.hidden)),
-                self.prefix + "up_proj.weight": TensorNeed((self.inter, self.hidden)),
-                self.prefix + "down_proj.weight": TensorNeed((self.hidden, self.inter))}
+        g, u, d = self.names
+        return {g: TensorNeed((self.inter, self.hidden)), u: TensorNeed((self.inter, self.hidden)), d: TensorNeed((self.hidden, self.inter))}
 
     def bind(self, get):
-        gate = to_compute(get(self.prefix + "gate_proj.weight"), self.dtype)
-        up = to_compute(get(self.prefix + "up_proj.weight"), self.dtype)
+        gate, up = (to_compute(get(n), self.dtype) for n in self.names[:2])
         # On the tensor-core path gate and up rows are interleaved in blocks of 16 and SiLU * up
         # happens in the product's epilogue; else they are stacked and a kernel of its own does it.
         self.fused = self.dtype == torch.bfloat16 and self.inter % 16 == 0 and self.hidden % 8 == 0
         self.gate_up = ops.bound_gemm(ops.interleave_gate_up(gate, up) if self.fused else torch.cat([gate, up], dim=0).contiguous(),
-                                      silu=self.fused)
+                                      silu=self.epilogue if self.fused else 0)
         del gate, up
-        self.down = ops.bound_gemm(to_compute(get(self.prefix + "down_proj.weight"), self.dtype).contiguous())
+        self.down = ops.bound_gemm(to_compute(get(self.names[2]), self.dtype).contiguous())
         self.w_gate_up, self.w_down = self.gate_up.w, self.down.w      # as the products keep them (in k-blocks when they stream them)
         self._partial_capacity = None
 
@@ -47,7 +54,10 @@ class SwiGLU(FeedForward):
         else:
             gu = ctx.ws.rows("ffn.gate_up", T, 2 * self.inter, self.dtype)
             self.gate_up(h, gu)
-            ops.silu_mul(gu, act)
+            if self.epilogue == ops.GATED_SILU:
+                ops.silu_mul(gu, act)
+            else:
+                ops.glu_biased(gu, None, None, act, ops.ACT_RELU)
         out = ctx.ws.rows("ffn.out", T, self.hidden, self.dtype)
         if self._partial_capacity is None:
             self._partial_capacity = ops.partial_capacity(ctx.ws.max_rows, self.down.N, self.down.K)
@@ -190,7 +200,32 @@ class TwoBranchMLP(FeedForward):
         return self.down(act, out, lambda n: ctx.ws.flat("ffn.out.partial", n, torch.float32, self._partial_capacity))
 
 
+class FeedForwardSum(FeedForward):
+    """Feed-forwards side by side on the same input, summed: routed experts beside a shared one that every token passes. The
+    sum is handed on as an `ops.ScaledSum`: the residual add that follows forms it in float32. Their outputs must lie in
+    buffers of their own. params: `parts` = [PartSpec of a feed-forward, ...]."""
+    launches_only = False
+
+    def __init__(self, spec, dtype, prefix: str = ""):
+        from .base import build_part
+        self.parts = tuple(build_part("feed_forward", ps, dtype, prefix=prefix) for ps in spec["parts"])
+
+    def needs(self):
+        n = {}
+        for p in self.parts:
+            n.update(p.needs())
+        return n
+
+    def bind(self, get):
+        for p in self.parts:
+            p.bind(get)
+
+    def forward(self, h, ctx):
+        return ops.ScaledSum([term for p in self.parts for term in ops.flat_terms(p.forward(h, ctx))])
+
+
 register_part("feed_forward", "swiglu", SwiGLU, replace=True)
+register_part("feed_forward", "feed_forward_sum", FeedForwardSum, replace=True)
 register_part("feed_forward", "two_branch_mlp", TwoBranchMLP, replace=True)
 register_part("feed_forward", "biased_glu", BiasedGLU, replace=True)
 register_part("feed_forward", "clamped_glu", ClampedGLU, replace=True)

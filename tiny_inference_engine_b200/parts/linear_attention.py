@@ -111,4 +111,78 @@ class GatedLinearAttention(Mixer):
         return self.gemm_o(gated, out, lambda m: ctx.ws.flat("mixer.out.partial", m, torch.float32, self._capacity))
 
 
+class ConstantDecayAttention(Mixer):
+    """Linear attention whose matrix state decays with one constant per head:
+
+        q, k, v = silu(h Wq^T), silu(h Wk^T), silu(h Wv^T)
+        S <- decay_h S + k v^T;   o = S^T q                        the read-out sees the token's own write; no other scale
+        out     = ((o / rms(o) over ALL heads together) * w_norm * sigmoid(h Wg^T)) Wo^T
+
+    S (float32 [dim, value_dim] per head, zero at the start of a sequence) is a request's state. The four projections are one
+    stacked product; everything behind them up to the gate is float32. params: `hidden_size`, `num_heads`, `head_dim`,
+    `value_dim`, `decay` (a number per head), `eps`."""
+    launches_only = False
+    graph_safe = True
+
+    def __init__(self, spec, dtype, prefix: str = ""):
+        p = spec.params
+        self.prefix = prefix + p.get("prefix", "")
+        self.hidden, self.heads = int(p["hidden_size"]), int(p["num_heads"])
+        self.dim, self.vdim = int(p["head_dim"]), int(p["value_dim"])
+        self.eps = float(p.get("eps", 1e-6))
+        self.decay_values = [float(d) for d in p["decay"]]
+        if min(self.heads, self.vdim) <= 0 or not 0 < self.dim <= 256 or len(self.decay_values) != self.heads:
+            raise InvalidArgument(f"constant-decay attention: bad sizes heads={self.heads} dim={self.dim} (1 to 256) vdim={self.vdim} "
+                                  f"with {len(self.decay_values)} decays")
+        self.dtype = dtype
+        self.nqk, self.nv = self.heads * self.dim, self.heads * self.vdim
+        self.q_off, self.k_off = 0, _up8(self.nqk)
+        self.v_off = self.k_off + _up8(self.nqk)
+        self.g_off = self.v_off + _up8(self.nv)
+        self.width = self.g_off + _up8(self.nv)
+        self.state_floats = self.heads * self.dim * self.vdim
+
+    def needs(self):
+        D, n = self.hidden, lambda leaf: self.prefix + leaf
+        return {n("q"): TensorNeed((self.nqk, D)), n("k"): TensorNeed((self.nqk, D)), n("v"): TensorNeed((self.nv, D)),
+                n("g"): TensorNeed((self.nv, D)), n("o"): TensorNeed((D, self.nv)), n("norm"): TensorNeed((self.nv,), "norm")}
+
+    def bind(self, get):
+        n = lambda leaf: self.prefix + leaf
+        stacked = torch.zeros((self.width, self.hidden), dtype=self.dtype, device=get(n("q")).device)
+        for leaf, off, rows in (("q", self.q_off, self.nqk), ("k", self.k_off, self.nqk), ("v", self.v_off, self.nv), ("g", self.g_off, self.nv)):
+            stacked[off:off + rows] = to_compute(get(n(leaf)), self.dtype)
+        self.gemm_in = ops.bound_gemm(stacked, split_many=False)
+        self.w_in = self.gemm_in.w
+        self.gemm_o = ops.bound_gemm(to_compute(get(n("o")), self.dtype).contiguous(), split_many=True)
+        self.w_o = self.gemm_o.w
+        self.norm_w = get(n("norm")).to(torch.float32).contiguous()
+        self.decay = torch.tensor([self.decay_values], dtype=torch.float32, device=self.norm_w.device)      # one row for every token
+        self._capacity = None
+
+    def state_need(self):
+        return StateNeed((self.state_floats,), torch.float32)
+
+    def forward(self, h, ctx, cache, state):
+        T, H, dim, vdim = h.shape[0], self.heads, self.dim, self.vdim
+        if state is None:
+            raise InvalidArgument("constant-decay attention needs state slots (make the cache with `make_cache`)")
+        proj = ctx.ws.rows("cda.proj", T, self.width, self.dtype)
+        self.gemm_in(h, proj)
+        qn = ctx.ws.rows("cda.q", T, self.nqk, torch.float32)
+        kn = ctx.ws.rows("cda.k", T, self.nqk, torch.float32)
+        vn = ctx.ws.rows("cda.v", T, self.nv, torch.float32)
+        ops.act_split(proj, self.q_off, self.k_off, self.v_off, qn, kn, vn)
+        o = ctx.ws.rows("cda.o", T, self.nv, torch.float32)
+        ops.delta_rule(qn, kn, vn, None, self.decay.expand(T, H), state, self.state_floats, proj, self.q_off, self.k_off, self.v_off,
+                       ctx.query_start, ctx.state_slots, ctx.S, H, H, dim, vdim, 1, o, plain=True, decay_per_head=True)
+        gated = ctx.ws.rows("cda.gated", T, self.nv, self.dtype)
+        ops.head_norm_gate(o, proj[:, self.g_off:self.g_off + self.nv], self.norm_w, self.eps, gated, 1, self.nv, ops.GATE_SIGMOID)
+        out = ctx.ws.rows("mixer.out", T, self.hidden, self.dtype)
+        if self._capacity is None:
+            self._capacity = ops.partial_capacity(ctx.ws.max_rows, self.gemm_o.N, self.gemm_o.K)
+        return self.gemm_o(gated, out, lambda m: ctx.ws.flat("mixer.out.partial", m, torch.float32, self._capacity))
+
+
 register_part("mixer", "gated_linear_attention", GatedLinearAttention, replace=True)
+register_part("mixer", "constant_decay_attention", ConstantDecayAttention, replace=True)

@@ -127,3 +127,39 @@ class DynamicTanh(Norm):
 
 
 register_part("norm", "dynamic_tanh", DynamicTanh, replace=True)
+
+
+class LayerNorm(Norm):
+    """A norm with mean and variance: (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias, the bias stored beside
+    the weight as `<name>.b`. The residual add ahead of it is fused in: a plain delta, the partial sums of a split product,
+    or a sum of up to four sublayer outputs with factors (`ops.ScaledSum`), all in float32."""
+    launches_only = False
+    takes_split_sum = True
+    takes_scaled_sum = True
+
+    def __init__(self, spec, dtype, prefix: str = ""):
+        self.name = prefix + spec["name"]
+        self.size = int(spec["size"])
+        self.eps = float(spec["eps"])
+        self.dtype = dtype
+        self.weight = self.bias = None
+
+    def needs(self):
+        return {self.name: TensorNeed((self.size,), "norm"), self.name + ".b": TensorNeed((self.size,), "norm")}
+
+    def bind(self, get):
+        self.weight = get(self.name).to(torch.float32).contiguous()
+        self.bias = get(self.name + ".b").to(torch.float32).contiguous()
+
+    def add_norm(self, x, delta, out, rows=None):
+        if isinstance(delta, ops.NormedDelta):
+            raise NotImplementedError("a layer norm takes a plain delta, partial sums or a scaled sum, not one that still has a norm to pass")
+        ops.add_layer_norm(x, delta, self.weight, self.bias, self.eps, out, rows)
+
+    def rows(self, x, out):
+        if x.dtype != torch.float32 or not x.is_contiguous():
+            raise NotImplementedError("a layer norm over other views than contiguous float32 rows")
+        ops.add_layer_norm(x, None, self.weight, self.bias, self.eps, out)
+
+
+register_part("norm", "layer_norm", LayerNorm, replace=True)

@@ -24,12 +24,20 @@ class RotaryEncoding(PositionEncoding):
         i = np.arange(self.rotary_dim // 2, dtype=np.float32)
         expo = (np.float32(2.0) * i) / np.float32(self.rotary_dim)
         self.inv_freq_host = (np.float32(1.0) / np.power(np.float32(self.theta), expo, dtype=np.float32)).astype(np.float32)
-        self._table = None
+        self._table = self._turns = None
 
     def fused_table(self):
         if self._table is None:
             self._table = torch.from_numpy(self.inv_freq_host).cuda()
         return self._table
+
+    def turns_table(self):
+        """float64 [rotary_dim / 2]: the turns a position makes, theta^(-2i/rotary_dim) / (2 pi). For kernels that form the
+        angle in double precision, so that far positions lose nothing."""
+        if self._turns is None:
+            i = np.arange(self.rotary_dim // 2, dtype=np.float64)
+            self._turns = torch.from_numpy(self.theta ** (-2.0 * i / self.rotary_dim) / (2.0 * np.pi)).cuda()
+        return self._turns
 
     def apply(self, x, positions, heads, head_dim):
         ops.rope(x, positions, self.fused_table(), heads, head_dim)

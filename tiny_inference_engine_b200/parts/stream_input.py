@@ -42,14 +42,17 @@ class ConcatProjection(StreamInput):
 
 class PassVector(StreamInput):
     """x[t] += vectors[index]: one learned vector joins every row of the stream (float32) ahead of a pass over a span
-    of layers; `vectors` is [passes, hidden] and every pass names its own row. params: `name`, `index`, `passes`,
-    `hidden_size`."""
+    of layers; `vectors` is [passes, hidden] and every pass names its own row. With `add_origin` the embedding part's
+    output joins the stream first, x[t] += origin[t]. The pending delta of the layer before (any sum of sublayer outputs)
+    is added ahead of both, all in float32. params: `name`, `index`, `passes`, `hidden_size`, `add_origin`."""
     launches_only = True
-    reads_origin = False        # the model need not keep the embedding's output for it
 
     def __init__(self, spec, dtype, prefix: str = ""):
         self.name = prefix + spec["name"]
         self.index, self.passes, self.hidden = int(spec["index"]), int(spec["passes"]), int(spec["hidden_size"])
+        self.add_origin = bool(spec.params.get("add_origin", False))
+        self.reads_origin = self.add_origin     # without it the model need not keep the embedding's output
+        self.dtype = dtype
         self.vector = None
 
     def needs(self):
@@ -59,9 +62,12 @@ class PassVector(StreamInput):
         self.vector = get(self.name)[self.index].to(torch.float32).contiguous()
 
     def forward(self, x, pending, origin, ctx):
-        if pending is not None:
-            raise NotImplementedError("pass_vector stands behind layers that leave the stream complete")
-        ops.add_row_vector(x, self.vector)
+        if isinstance(pending, ops.NormedDelta):
+            raise NotImplementedError("pass_vector takes a plain delta, partial sums or a scaled sum, not one that still has a norm to pass")
+        if pending is None and not self.add_origin:
+            ops.add_row_vector(x, self.vector)
+        else:
+            ops.stream_add(x, pending, self.dtype, other=origin if self.add_origin else None, vec=self.vector)
         return None
 
 

@@ -104,8 +104,9 @@ class TokenShiftRecurrence(Mixer):
 
 class MixerSum(Mixer):
     """Mixers side by side on the same input, summed with one factor each: sum_i scale_i * mixer_i(h). At most one of them
-    keeps pages and at most one keeps state, which become this mixer's own. The sum is handed on as an `ops.ScaledSum`:
-    the residual add that follows forms it in float32. params: `parts` = [(PartSpec of a mixer, factor), ...] (two)."""
+    keeps pages, which become this mixer's own; the float32 rows of state that they keep lie one behind the other in this
+    mixer's row, each starting on a 16-byte boundary. The sum is handed on as an `ops.ScaledSum`: the residual add that
+    follows forms it in float32. params: `parts` = [(PartSpec of a mixer, factor), ...] (two)."""
     launches_only = False
 
     def __init__(self, spec, dtype, prefix: str = ""):
@@ -113,9 +114,17 @@ class MixerSum(Mixer):
         self.parts = [(build_part("mixer", ps, dtype, prefix=prefix), float(c)) for ps, c in spec["parts"]]
         if len(self.parts) != 2:
             raise InvalidArgument(f"a sum of mixers has two of them, got {len(self.parts)}")
-        if sum(m.cache_need() is not None for m, _ in self.parts) > 1 or sum(m.state_need() is not None for m, _ in self.parts) > 1:
-            raise InvalidArgument("a sum of mixers: at most one of them keeps pages and at most one keeps state")
+        if sum(m.cache_need() is not None for m, _ in self.parts) > 1:
+            raise InvalidArgument("a sum of mixers: at most one of them keeps pages")
         self.mixers = tuple(m for m, _ in self.parts)
+        needs = [m.state_need() for m in self.mixers]
+        if sum(n is not None for n in needs) > 1 and any(n is not None and (len(n.shape) != 1 or n.dtype != torch.float32) for n in needs):
+            raise InvalidArgument("a sum of mixers that keep state takes float32 rows of state")
+        self.state_at, at = [], 0       # each mixer's columns of the row; None: it keeps none
+        for n in needs:
+            self.state_at.append(None if n is None else (at, at + n.shape[0]))
+            at += 0 if n is None else (n.shape[0] + 3) // 4 * 4
+        self.state_floats = at
         self.graph_safe = all(m.graph_safe for m in self.mixers if m.state_need() is not None)
 
     def needs(self):
@@ -132,11 +141,16 @@ class MixerSum(Mixer):
         return next((m.cache_need() for m in self.mixers if m.cache_need() is not None), None)
 
     def state_need(self):
-        return next((m.state_need() for m in self.mixers if m.state_need() is not None), None)
+        needs = [m.state_need() for m in self.mixers if m.state_need() is not None]
+        if len(needs) <= 1:
+            return needs[0] if needs else None
+        return StateNeed((self.state_floats,), torch.float32)
 
     def forward(self, h, ctx, cache, state):
+        alone = sum(at is not None for at in self.state_at) <= 1
         return ops.ScaledSum([(m.forward(h, ctx, cache if m.cache_need() is not None else None,
-                                         state if m.state_need() is not None else None), c) for m, c in self.parts])
+                                         None if at is None or state is None else (state if alone else state[:, at[0]:at[1]])), c)
+                              for (m, c), at in zip(self.parts, self.state_at)])
 
 
 register_part("mixer", "token_shift_recurrence", TokenShiftRecurrence, replace=True)
