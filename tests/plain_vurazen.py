@@ -318,3 +318,168 @@ def generate(w, cfg, prompt, n):
     for _ in range(n):
         toks.append(int(np.argmax(forward(w, cfg, toks)[-1])))
     return toks[len(prompt):]
+
+
+# --------------------------------------------------------------------------- configurations and weights for the tests
+
+def dense(ff=72):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(ff=24, experts=6, top=2, limit=1.5, shared_ff=20, shared_limit=1.0):
+    return {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "top": top},
+            "shared": {"ff": shared_ff, "limit": shared_limit}}
+
+
+def scan_layer(inner=48, state=12, dt_rank=5, conv=4, mlp="dense"):
+    return {"type": "mamba1", "mixer": {"inner": inner, "state": state, "dt_rank": dt_rank, "conv": conv}, "mlp": dense() if mlp == "dense" else mlp}
+
+
+def parallel_layer(heads=4, kv_heads=2, dim=16, window=20, keep_first=3, softcap=20.0, scale=None, rot=8, base=10000.0, conv=4, rheads=4,
+                   rkv_heads=2, rdim=12, rvdim=20, rconv=4, left_scale=0.7, right_scale=1.2, mlp="dense"):
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": conv, "softcap": softcap,
+            "scale": float(scale if scale is not None else dim ** -0.5), "mask": {"size": window, "keep_first": keep_first},
+            "rot": {"base": base, "dims": rot}}
+    right = {"heads": rheads, "kv_heads": rkv_heads, "dim": rdim, "vdim": rvdim, "conv": rconv}
+    return {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": left_scale, "right_scale": right_scale},
+            "mlp": dense() if mlp == "dense" else mlp}
+
+
+def lightning_layer(heads=3, dim=12, vdim=20, decay=None, mlp="dense"):
+    decay = [float(d) for d in (decay if decay is not None else np.exp(-np.exp(np.linspace(-0.5, -6.0, heads))))]
+    return {"type": "lightning", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay}, "mlp": dense() if mlp == "dense" else mlp}
+
+
+def make_config(layers, vocab=160, width=64, eps=1e-5, scale=3.0, softcap=25.0, loop=None):
+    cfg = {"architecture": "Vurazen", "embedding": {"scale": scale}, "layers": layers, "logit_softcap": softcap, "norm": {"eps": eps},
+           "vocab": vocab, "width": width}
+    if loop is not None:
+        cfg["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return cfg
+
+
+def tensor_shapes(cfg, ranks=(6, 10)):
+    """ranks: the inner sizes of a right mixer's decay and gate projections."""
+    D = cfg["width"]
+    s = {"embed": (cfg["vocab"], D), "head": (cfg["vocab"], D)}
+    if cfg.get("loop"):
+        s["loop.step"] = (cfg["loop"]["times"], D)
+
+    def norm(name):
+        s[name], s[name + ".b"] = (D,), (D,)
+
+    for i, layer in enumerate(cfg["layers"]):
+        p, mx = f"l{i}.", layer["mixer"]
+        norm(p + "norm1")
+        m = p + "mix."
+        if layer["type"] == "mamba1":
+            I, N, r = mx["inner"], mx["state"], mx["dt_rank"]
+            s[m + "in"], s[m + "conv"], s[m + "conv.b"] = (2 * I, D), (I, mx["conv"]), (I,)
+            s[m + "x"], s[m + "dt"], s[m + "dt.b"] = (r + 2 * N, I), (I, r), (I,)
+            s[m + "A_log"], s[m + "D"], s[m + "o"] = (I, N), (I,), (D, I)
+        elif layer["type"] == "lightning":
+            nqk, nv = mx["heads"] * mx["dim"], mx["heads"] * mx["vdim"]
+            s[m + "q"], s[m + "k"], s[m + "v"], s[m + "g"], s[m + "o"], s[m + "norm"] = (nqk, D), (nqk, D), (nv, D), (nv, D), (D, nv), (nv,)
+        else:
+            lf, rt = mx["left"], mx["right"]
+            a, nq, nk = m + "left.", lf["heads"] * lf["dim"], lf["kv_heads"] * lf["dim"]
+            s[a + "q"], s[a + "k"], s[a + "q.b"], s[a + "k.b"] = (nq, D), (nk, D), (nq,), (nk,)
+            s[a + "q.conv"], s[a + "k.conv"] = (nq, lf["conv"]), (nk, lf["conv"])
+            s[a + "sink"], s[a + "o"] = (lf["heads"],), (D, nq)
+            b, H, dim, vdim = m + "right.", rt["heads"], rt["dim"], rt["vdim"]
+            nqk, nv = rt["kv_heads"] * dim, H * vdim
+            for leaf, n in (("q", nqk), ("k", nqk), ("v", nv)):
+                s[b + leaf], s[b + leaf + ".conv"] = (n, D), (n, rt["conv"])
+            s[b + "b"], s[b + "A_log"], s[b + "norm"] = (H, D), (H,), (vdim,)
+            s[b + "a1"], s[b + "a2"], s[b + "dt_bias"] = (ranks[0], D), (H * dim, ranks[0]), (H * dim,)
+            s[b + "g1"], s[b + "g2"], s[b + "o"] = (ranks[1], D), (nv, ranks[1]), (D, nv)
+        mlp = layer.get("mlp")
+        if mlp is not None:
+            q = p + "mlp."
+            units = [q] if mlp["kind"] == "dense" else [f"{q}e{e}." for e in range(mlp["router"]["experts"])]
+            ff = mlp["ff"] if mlp["kind"] == "dense" else mlp["expert"]["ff"]
+            sizes = [(u, ff) for u in units]
+            if mlp["kind"] == "moe":
+                s[q + "router"], s[q + "router.b"] = (mlp["router"]["experts"], D), (mlp["router"]["experts"],)
+                sizes.append((q + "shared.", mlp["shared"]["ff"]))
+            for u, n in sizes:
+                s[u + "gate"], s[u + "up"], s[u + "down"] = (n, D), (n, D), (D, n)
+    norm("final.norm")
+    return s
+
+
+def random_weights(cfg, seed, ranks=(6, 10), sharp=3.0, expert_gain=1.0):
+    """float32 weights that bfloat16 holds exactly (so that both dtypes load the same model). Matrices are N(0, 1/in);
+    attention's queries and keys are `sharp` times larger so that attention is not flat and a key that is lost or misplaced
+    moves the logits; decays and step sizes are spread between fast and slow channels. `expert_gain` scales what the routed
+    experts add: a router's close call that 16-bit rounding decides the other way then stays inside a 16-bit tolerance."""
+    rng = np.random.default_rng(seed)
+    w = {}
+    for name, shape in tensor_shapes(cfg, ranks).items():
+        leaf = name.split(".")[-1]
+        if name == "embed":
+            t = rng.standard_normal(shape)
+        elif name == "loop.step":
+            t = rng.standard_normal(shape) * 0.7
+        elif leaf in ("norm1", "norm"):
+            t = 1.0 + rng.standard_normal(shape) * 0.1
+        elif name.endswith("right.b"):
+            t = rng.standard_normal(shape) / np.sqrt(shape[-1])
+        elif name.endswith("dt.b"):
+            t = rng.uniform(-6.0, 0.5, shape)
+        elif name.endswith("router.b"):
+            t = rng.standard_normal(shape)
+        elif leaf == "b":
+            t = rng.standard_normal(shape) * 0.3
+        elif leaf == "conv":
+            t = rng.standard_normal(shape) * 0.5
+            t[:, -1] += 0.7
+        elif leaf == "sink":
+            t = rng.uniform(-1.0, 3.0, shape)
+        elif leaf == "A_log":
+            t = rng.uniform(-2.0, 1.5, shape)
+        elif leaf == "dt_bias":
+            t = rng.uniform(-5.0, 0.5, shape)
+        elif leaf == "D":
+            t = rng.standard_normal(shape)
+        else:
+            t = rng.standard_normal(shape) / np.sqrt(shape[-1])
+            if leaf in ("q", "k") and ".left." in name:
+                t = t * sharp
+            if leaf == "router":
+                t = t * 3.0
+            if leaf == "down" and ".mlp.e" in name:
+                t = t * expert_gain
+        w[name] = round_bf16(np.asarray(t, dtype=np.float32))
+    return w
+
+
+def write_safetensors(path, tensors, bf16=True):
+    """One file: 8-byte little-endian header length, JSON header, data. bf16 stores the upper 16 bits."""
+    header, blobs, off = {}, [], 0
+    for name, t in tensors.items():
+        shape = list(np.shape(t))
+        a = np.ascontiguousarray(t, dtype=np.float32).reshape(-1)
+        if bf16:
+            data = (a.view(np.uint32) >> 16).astype("<u2").tobytes()
+            dt = "BF16"
+        else:
+            data = a.astype("<f4").tobytes()
+            dt = "F32"
+        header[name] = {"dtype": dt, "shape": shape, "data_offsets": [off, off + len(data)]}
+        blobs.append(data)
+        off += len(data)
+    hj = json.dumps(header).encode()
+    hj += b" " * (-len(hj) % 8)
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(hj)))
+        f.write(hj)
+        for b in blobs:
+            f.write(b)
+
+
+def write_model_dir(path, cfg, weights, bf16=True):
+    path = Path(path)
+    path.mkdir(parents=True, exist_ok=True)
+    (path / "config.json").write_text(json.dumps(cfg))
+    write_safetensors(path / "model.safetensors", weights, bf16=bf16)

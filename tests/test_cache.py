@@ -10,6 +10,7 @@ from tiny_inference_engine_b200.parts import CacheNeed, StateNeed
 
 FULL = CacheNeed("full", 2, 16)
 WIN = CacheNeed("window", 1, 32, window=20)
+KEPT = CacheNeed("window", 1, 32, window=20, keep_first=9)
 
 
 def test_pool_lowest_first_reuse_and_misuse():
@@ -89,6 +90,36 @@ def test_window_group_gives_pages_back_as_the_window_passes():
     assert m.num_free(0) == 12 and m.num_free(1) == 12
 
 
+def test_a_window_group_keeps_the_pages_of_the_first_tokens():
+    m = CacheManager([WIN, KEPT], page_size=8, num_pages=12)
+    assert len(m.groups) == 2 and m.groups[1].keep_first == 9          # not the group of the same window without kept tokens
+    r = m.new_request()
+    assert m.reserve(r, 64)
+    first = list(r.tables[1].view()[:2])
+    m.advance_window(r, 28)     # the next query reads keys from 9 on: page 0 is passed, but holds kept tokens
+    assert r.tables[0].released == 1 and m.num_free(0) == 5 and m.num_free(1) == 4
+    m.advance_window(r, 64)     # from 45 on: pages 0..4 are passed; tokens 0..8 are in pages 0 and 1
+    win, kept = r.tables
+    assert list(win.view()[:5]) == [FREED] * 5 and m.num_free(0) == 9
+    assert list(kept.view()[:2]) == first and list(kept.view()[2:5]) == [FREED] * 3 and m.num_free(1) == 7
+    assert sorted(kept.held()) == sorted(first + [int(b) for b in kept.view()[5:]])
+    m.reset(r)                  # preemption gives the kept pages back too
+    assert not m.holds(r) and m.num_free(1) == 12
+    assert m.reserve(r, 5) and m.holds(r)
+    m.advance_window(r, 5)
+    m.release(r)
+    assert m.num_free(0) == 12 and m.num_free(1) == 12
+    # a bounded group has room for the kept pages beside the window's
+    b = CacheManager([FULL, KEPT], page_size=8, num_pages=100, window_requests=2, window_step_tokens=12)
+    assert b.group_pages == [100, 2 * (4 + 2 + 2)]
+    for at in range(12, 400, 12):
+        r = r if at > 12 else b.new_request()
+        assert b.reserve(r, at)
+        b.advance_window(r, at)
+        assert b.group_pages[1] - b.num_free(1) <= 8
+    b.release(r)
+
+
 def test_a_state_slot_is_taken_by_the_first_reserve_and_given_back_by_reset_and_release():
     states = StateSlots([None, StateNeed((4,))], max_requests=2)
     m = CacheManager([FULL, None], page_size=4, num_pages=6, state_slots=states)
@@ -147,8 +178,8 @@ def test_a_window_group_gets_the_pages_it_can_use_and_the_budget_goes_to_the_res
 def test_no_page_is_lost_held_twice_or_freed_twice_under_random_orders(seed):
     rng = random.Random(seed)
     page = rng.choice([4, 8, 16])
-    states = StateSlots([StateNeed((2,)), None, None], max_requests=rng.randint(2, 6))
-    m = CacheManager([FULL, WIN, FULL], page_size=page, num_pages=rng.randint(6, 40), state_slots=states,
+    states = StateSlots([StateNeed((2,)), None, None, None], max_requests=rng.randint(2, 6))
+    m = CacheManager([FULL, WIN, FULL, KEPT], page_size=page, num_pages=rng.randint(6, 40), state_slots=states,
                      window_requests=rng.choice([None, 2, 6]), window_step_tokens=3 * page)
     live = {}   # request -> tokens covered
     for _ in range(400):

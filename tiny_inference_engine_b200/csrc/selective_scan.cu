@@ -41,6 +41,26 @@ __device__ __forceinline__ float ex2(float v) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
   return r;
 }
+// 2^v for v <= 0 to half a unit in the last place and without a bias: a slow channel multiplies thousands of decays that are
+// all close to one, and an approximation that errs to one side there shows in the float32 path. 2^v = 2^n e^(f ln 2) with n
+// the nearest integer; |f ln 2| <= 0.347, where the exponential series to the seventh power leaves 5e-9.
+__device__ __forceinline__ float ex2_precise(float v) {
+  const float n = rintf(v), r = (v - n) * 0.69314718055994531f;
+  float p = 1.0f / 5040.0f;
+  p = fmaf(p, r, 1.0f / 720.0f);
+  p = fmaf(p, r, 1.0f / 120.0f);
+  p = fmaf(p, r, 1.0f / 24.0f);
+  p = fmaf(p, r, 1.0f / 6.0f);
+  p = fmaf(p, r, 0.5f);
+  p = fmaf(p, r, 1.0f);
+  p = fmaf(p, r, 1.0f);
+  return v < -125.0f ? 0.0f : p * __int_as_float((static_cast<int>(n) + 127) << 23);
+}
+template <typename T>
+__device__ __forceinline__ float decay_ex2(float v) {
+  if constexpr (sizeof(T) == 4) return ex2_precise(v);
+  else return ex2(v);
+}
 __device__ __forceinline__ void scan_copy16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))), "l"(src) : "memory");
 }
@@ -176,7 +196,7 @@ __global__ void __launch_bounds__(LANES * kScanChannels) selective_scan_kernel(S
           const float* ct = cs + (tb + q) * L.np + lane * R;
 #pragma unroll
           for (int r = 0; r < R; ++r) {
-            sr[r] = fmaf(ex2(d.x * ar[r]), sr[r], d.y * bt[r]);
+            sr[r] = fmaf(decay_ex2<T>(d.x * ar[r]), sr[r], d.y * bt[r]);
             y[q] = fmaf(sr[r], ct[r], y[q]);
           }
         }
