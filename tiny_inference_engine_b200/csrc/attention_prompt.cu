@@ -52,8 +52,19 @@ __device__ __forceinline__ int prompt_first_visible(int pos, int window, int chu
   return window > 0 ? max(0, pos - window + 1) : 0;
 }
 
+__device__ __forceinline__ float fast_exp2(float v) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+  return r;
+}
+__device__ __forceinline__ float fast_rcp(float v) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+  return r;
+}
+
 template <int DH, int STAGES>
-__global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const __grid_constant__ CUtensorMap k_map,
+__global__ void __launch_bounds__(kPromptThreads, DH <= 128 ? 2 : 1) attn_prompt_tma_kernel(const __grid_constant__ CUtensorMap k_map,
                                                                          const __grid_constant__ CUtensorMap v_map, PromptArgs a) {
   pdl_sync();
   using L = HalfLayout<DH>;
@@ -80,7 +91,7 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
   const int last_row = min(rows, row0 + 64) - 1;
   const int hi_cta = pos0 + last_row / G;
   const bool limited = a.window > 0 || a.chunk > 0;               // rows do not see all earlier keys
-  const bool shaped = a.softcap > 0.0f || a.r1 != nullptr;        // scores pass a cap or a bias: no tile is taken whole
+  const bool shaped = a.softcap > 0.0f || a.r1 != nullptr;        // scores pass a cap or a bias
   const int lo_cta = prompt_first_visible(pos0 + row0 / G, a.window, a.chunk);
   const int cache_heads = a.cache_heads > 0 ? a.cache_heads : a.kv_heads;
   const int cached_head = kvh % cache_heads, k_col = (kvh / cache_heads) * DH;
@@ -164,6 +175,7 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
     }
     const float scale = a.scale_log2 * 0.6931471805599453f;
     const float inv_cap = a.softcap > 0.0f ? 1.0f / a.softcap : 0.0f;
+    const float cap_in = 2.0f * a.scale_log2 * inv_cap, cap_log2 = a.softcap * 1.4426950408889634f;
     const bool warp_has_rows = row0 + warp * 16 < rows;
     const int warp_hi = warp_has_rows ? pos0 + min(rows - 1, row0 + warp * 16 + 15) / G : -1;   // largest position of the warp's rows
     const int warp_lo = warp_has_rows ? pos0 + (row0 + warp * 16) / G : -1;                     // smallest
@@ -184,13 +196,19 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
         for (int j = 0; j < 8; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.0f;
         qk_tile<DH, 8, L>(sc, qf, k_tile, 0);
         // no mask where every key of the tile is at or below every row's position and inside every row's window
-        const bool full_tile = !shaped && row0 + warp * 16 + 15 < rows && key0 + 63 <= warp_lo &&
+        const bool full_tile = a.r1 == nullptr && row0 + warp * 16 + 15 < rows && key0 + 63 <= warp_lo &&
                                (!limited || key0 + 63 < a.keep_first || key0 >= prompt_first_visible(warp_hi, a.window, a.chunk));
-        if (full_tile) {
+        if (full_tile && !shaped) {
 #pragma unroll
           for (int j = 0; j < 8; ++j) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) sc[j][e] *= a.scale_log2;
+          }
+        } else if (full_tile) {                // a cap alone: c tanh(s / c) = c - 2 c / (exp(2 s / c) + 1), in units of log2
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sc[j][e] = fmaf(-2.0f * cap_log2, fast_rcp(fast_exp2(sc[j][e] * cap_in) + 1.0f), cap_log2);
           }
         } else {
 #pragma unroll
@@ -201,7 +219,9 @@ __global__ void __launch_bounds__(kPromptThreads) attn_prompt_tma_kernel(const _
               const int pos = row_pos[e >> 1];
               const bool ok = key <= pos && (key >= row_lo[e >> 1] || key < a.keep_first);
               float v = sc[j][e] * a.scale_log2;
-              if (shaped && ok) {
+              if (shaped && ok && a.r1 == nullptr) {
+                v = fmaf(-2.0f * cap_log2, fast_rcp(fast_exp2(sc[j][e] * cap_in) + 1.0f), cap_log2);
+              } else if (shaped && ok) {
                 v = sc[j][e] * scale;
                 // float arithmetic on the fast exponential and logarithm (absolute error about 1e-6 of a score, far below what the
                 // bfloat16 products of this kernel carry): tanh(z) = 1 - 2 / (exp(2 z) + 1); ln(1 + x) with x >= 0

@@ -14,9 +14,8 @@
 //                head; further blocks turn the raw decay projection into decays (in place) and take beta's sigmoid.
 //   delta_rule   one block per (sequence, head, 16 columns): the recurrence over the sequence's tokens of the
 //                step, state read from and written back to the slot in row pieces through shared memory. Eight
-//                lanes share a column, each holding every eighth key channel; a chunk of tokens is staged in shared
-//                memory at a time. The blocks of a sequence also move the convolution's last inputs into the
-//                slot, a slice of the channels each.
+//                lanes share a column; a chunk of tokens is staged in shared memory at a time. The blocks of a
+//                sequence also move the convolution's last inputs into the slot, a slice of the channels each.
 //   delta_out    one warp per (token, head): o / rms(o) * w * sigmoid(gate).
 //
 // A state slot is one float row: S of every head [heads, dim, vdim], then the convolution's last taps - 1
@@ -112,24 +111,33 @@ __device__ __forceinline__ void async_copy16(float* dst, const float* src) {
 }
 __device__ __forceinline__ void async_copies_done() { asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory"); }
 
-constexpr int kDeltaCols = 16;       // columns of S that a block holds (LANES threads each)
+constexpr int kDeltaCols = 16;       // columns of S that a block holds
+constexpr int kDeltaLanes = 8;       // lanes of a warp that share a column
+constexpr int kDeltaThreads = kDeltaCols * kDeltaLanes;
 constexpr int kDeltaPad = kDeltaCols + 1;
+constexpr int kDeltaBatch = 4;       // tokens whose read-outs are summed over the lanes together
 
-// The key channel that register r of lane `lane` (of the LANES that share a column) holds: four channels in a row,
-// then the next four 32 channels on, so that a lane reads its k, q and decay entries 16 bytes at a time.
-template <int LANES>
-__device__ __forceinline__ int delta_row(int r, int lane) { return (r >> 2) * (4 * LANES) + lane * 4 + (r & 3); }
+// The key channel that register r of lane `lane` (of the eight that share a column) holds: four channels in a row, then the
+// next four 32 channels on, so that a lane reads its k, q and decay entries 16 bytes at a time and the lanes of a column
+// read 128 bytes in a row (the four columns of a warp read the same 128 bytes).
+__device__ __forceinline__ int delta_row(int r, int lane) { return (r >> 2) * (4 * kDeltaLanes) + lane * 4 + (r & 3); }
 
-// One block per (sequence, head, 16 columns of S). A column's key channels are spread over LANES lanes of a warp
-// (8, 16 or 32, by the head size: more lanes mean more warps to hide each other's latencies and fewer registers
-// each), so a token costs one pass over the registers with two dot products (against k and
-// against q of the decayed state, and k . q beside them), three shuffle steps for the three, and the update: with
-// d1 = (gS)^T k and d2 = (gS)^T q, u = beta (v - d1) and the read-out of the updated state is o = d2 + (k . q) u.
-// RMAX: key channels a lane may hold (dim <= LANES * RMAX).
-// BONUS (a specialization of the plain mode): the token reads the state as the token before left it and sees its own
-// write through a weight per key channel, o = S^T q + (sum_c bonus[h, c] k_c q_c) u, and only then S <- diag(decay) S + k u^T.
-template <typename T, int RMAX, int LANES, bool PLAIN, bool BONUS = false>
-__global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
+// What the recurrence does with a token (u is what it writes along its key):
+//   kDeltaRule   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   kDeltaPlain  S <- diag(g) S + k u^T, u = beta v;  o = S^T q
+//   kDeltaBonus  o = S^T q + (sum_c bonus[h, c] k_c q_c) u, u = beta v: the token reads the state as the token before left it
+//                and sees its own write through a weight per key channel;  then S <- diag(g) S + k u^T
+enum DeltaMode { kDeltaRule, kDeltaPlain, kDeltaBonus };
+
+// One block per (sequence, head, 16 columns of S). A column's key channels are spread over eight lanes, R a lane. What bounds
+// the kernel is the chain from token to token: in the delta rule a product over the lane's channels, three exchanges and the
+// update; without the correction the update alone. So everything else is kept off that chain and off the shared-memory pipe:
+// a column has few lanes (three exchanges instead of five, and one read of k, q and g serves the four columns of a warp), the
+// read-outs of four tokens are summed over the lanes together (each exchange halves the tokens that a lane still holds), and
+// k . q of a token is formed once a chunk, for all columns. In the delta rule the read-out of the updated state is
+// (gS)^T q + (k . q) u, so it does not wait for the update.
+template <typename T, int R, DeltaMode MODE>
+__global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(
     const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ vn, const float* __restrict__ beta,
     const float* __restrict__ decay, long long decay_stride, float* __restrict__ state, long long state_stride,
     long long conv_state_off, const T* __restrict__ proj, long long proj_stride, int q_off, int k_off, int v_off,
@@ -137,8 +145,8 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
     float* __restrict__ out, int decay_per_head, const float* __restrict__ bonus = nullptr) {
   // A block is one long chain of dependent steps, and there are few blocks (sequences x heads x column tiles). Started early
   // (programmatic dependent launch), beside a kernel that still fills the GPU, the blocks were placed on the few SMs that had
-  // room first and shared them: 1.7 instead of 0.6 ms for 2,048 tokens. So the launcher starts this kernel only when the
-  // kernels ahead have drained (launch_kernel_alone), and the kernel behind is let in when the walk over the tokens is done.
+  // room first and shared them. So for steps with portions the launcher starts this kernel only when the kernels ahead have
+  // drained (launch_kernel_alone), and the kernel behind is let in when the walk over the tokens is done.
   pdl_wait();
   extern __shared__ float smem[];
   const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * kDeltaCols;
@@ -147,26 +155,33 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
   const int t0 = query_start[s], n = query_start[s + 1] - t0;
   const int dim = sh.dim, vdim = sh.vdim, nqk = sh.kv_heads * dim, nv = sh.heads * vdim;
   const int g = h / (sh.heads / sh.kv_heads);
-  const int lane8 = threadIdx.x % LANES, cidx = threadIdx.x / LANES, col = col0 + cidx;      // lane8: the lane among those of its column
+  const int lane8 = threadIdx.x % kDeltaLanes, cidx = threadIdx.x / kDeltaLanes, col = col0 + cidx;
   const bool live = col < vdim;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* S = state + slot * state_stride + static_cast<long long>(h) * dim * vdim;
-  // The block's 16 columns of S come in row pieces of 64 bytes through shared memory (the lanes' own elements
-  // are a row apart in memory).
-  for (int i = threadIdx.x; i < dim * kDeltaCols; i += blockDim.x) {
-    const int r = i / kDeltaCols, c = i % kDeltaCols;
-    smem[r * kDeltaPad + c] = col0 + c < vdim ? S[static_cast<long long>(r) * vdim + col0 + c] : 0.0f;
-  }
-  __syncthreads();
-  float sreg[RMAX];
+  float* stage = smem;                        // the block's 16 columns of S on their way in and out, rows of kDeltaPad
+  const bool quads = vdim % 4 == 0 && (reinterpret_cast<uintptr_t>(S) & 15) == 0;
+  if (quads) {
+#pragma unroll 4
+    for (int i = threadIdx.x; i < dim * (kDeltaCols / 4); i += kDeltaThreads) {
+      const int r = i / (kDeltaCols / 4), c = (i % (kDeltaCols / 4)) * 4;
+      float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      if (col0 + c < vdim) load4(S + static_cast<long long>(r) * vdim + col0 + c, v);
 #pragma unroll
-  for (int r = 0; r < RMAX; ++r) {
-    const int rowi = delta_row<LANES>(r, lane8);
-    sreg[r] = rowi < dim ? smem[rowi * kDeltaPad + cidx] : 0.0f;
+      for (int e = 0; e < 4; ++e) stage[r * kDeltaPad + c + e] = v[e];
+    }
+  } else {
+    for (int i = threadIdx.x; i < dim * kDeltaCols; i += kDeltaThreads) {
+      const int r = i / kDeltaCols, c = i % kDeltaCols;
+      stage[r * kDeltaPad + c] = col0 + c < vdim ? S[static_cast<long long>(r) * vdim + col0 + c] : 0.0f;
+    }
   }
   // Chunks of tokens come through two buffers in turn: while one is worked on, asynchronous copies fill the other.
-  // A buffer: k [chunk][dim], q [chunk][dim], decays [chunk][dim], v [chunk][kDeltaCols], beta [chunk].
-  const int buf_floats = (chunk * (3 * dim + kDeltaCols + 1) + 3) & ~3;      // a buffer starts on a 16-byte boundary
+  // A buffer: k [chunk][dim], q [chunk][dim], decays [chunk][dim] (or [chunk]), v [chunk][kDeltaCols], beta [chunk].
+  float* const buffers = smem + ((dim * kDeltaPad + 3) & ~3);
+  const int g_ld = decay_per_head ? 1 : dim;
+  const int buf_floats = (chunk * (2 * dim + g_ld + kDeltaCols + 1) + 3) & ~3;      // a buffer starts on a 16-byte boundary
+  float* const kq = buffers + 2 * buf_floats;                                       // [chunk]: k . q of the chunk's tokens
   const bool vec4 = dim % 4 == 0;
   const bool wide = vec4 && nqk % 4 == 0 && ((reinterpret_cast<uintptr_t>(kn) | reinterpret_cast<uintptr_t>(qn)) & 15) == 0 &&
                     (decay_per_head || (decay_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(decay) & 15) == 0));
@@ -175,11 +190,10 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
     float* kb = base;
     float* qb = kb + chunk * dim;
     float* gb = qb + chunk * dim;
-    float* vb = gb + chunk * dim;
-    float* bb = vb + chunk * kDeltaCols;
+    float* bb = gb + chunk * g_ld + chunk * kDeltaCols;
     if (wide) {
       const int pieces = dim / 4;
-      for (int i = threadIdx.x; i < cn * pieces; i += blockDim.x) {
+      for (int i = threadIdx.x; i < cn * pieces; i += kDeltaThreads) {
         const int tc = i / pieces, d = (i % pieces) * 4;
         const long long t = t0 + c0 + tc;
         async_copy16(kb + tc * dim + d, kn + t * nqk + g * dim + d);
@@ -187,7 +201,7 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
         if (!decay_per_head) async_copy16(gb + tc * dim + d, decay + t * decay_stride + h * dim + d);
       }
     } else {
-      for (int i = threadIdx.x; i < cn * dim; i += blockDim.x) {
+      for (int i = threadIdx.x; i < cn * dim; i += kDeltaThreads) {
         const int tc = i / dim, d = i % dim;
         const long long t = t0 + c0 + tc;
         async_copy4(kb + i, kn + t * nqk + g * dim + d);
@@ -195,116 +209,158 @@ __global__ void __launch_bounds__(LANES * kDeltaCols) delta_rule_kernel(
         if (!decay_per_head) async_copy4(gb + i, decay + t * decay_stride + h * dim + d);
       }
     }
-    for (int i = threadIdx.x; i < cn * kDeltaCols; i += blockDim.x) {
+    float* vb = gb + chunk * g_ld;
+    for (int i = threadIdx.x; i < cn * kDeltaCols; i += kDeltaThreads) {
       const int tc = i / kDeltaCols, c = col0 + i % kDeltaCols;
       if (c < vdim) async_copy4(vb + i, vn + (t0 + c0 + tc) * static_cast<long long>(nv) + h * vdim + c);
       else vb[i] = 0.0f;
     }
-    if (decay_per_head)                       // one factor a token and head: at the start of the token's row
-      for (int i = threadIdx.x; i < cn; i += blockDim.x) async_copy4(gb + i * dim, decay + (t0 + c0 + i) * decay_stride + h);
-    for (int i = threadIdx.x; i < cn; i += blockDim.x) {
+    for (int i = threadIdx.x; i < cn; i += kDeltaThreads) {
+      if (decay_per_head) async_copy4(gb + i, decay + (t0 + c0 + i) * decay_stride + h);
       if (beta) async_copy4(bb + i, beta + (t0 + c0 + i) * static_cast<long long>(sh.heads) + h);
       else bb[i] = 1.0f;
     }
   };
-  __syncthreads();                            // the staging tile above is done with: the buffers lie over it
-  fetch(0, smem);
+  fetch(0, buffers);
+  __syncthreads();
+  float sreg[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int rowi = delta_row(r, lane8);
+    sreg[r] = rowi < dim ? stage[rowi * kDeltaPad + cidx] : 0.0f;
+  }
   int turn = 0;
   for (int c0 = 0; c0 < n; c0 += chunk, turn ^= 1) {
     const int cn = min(chunk, n - c0);
-    float* base = smem + turn * buf_floats;
-    const float* kb = base;
+    const float* kb = buffers + turn * buf_floats;
     const float* qb = kb + chunk * dim;
     const float* gb = qb + chunk * dim;
-    const float* vb = gb + chunk * dim;
+    const float* vb = gb + chunk * g_ld;
     const float* bb = vb + chunk * kDeltaCols;
     async_copies_done();
     __syncthreads();                          // this chunk is there, and everyone is through with the other buffer
-    if (c0 + chunk < n) fetch(c0 + chunk, smem + (turn ^ 1) * buf_floats);
-    float* kq = smem + 2 * buf_floats;        // [chunk <= 16]
-    if (PLAIN) {
-      // k . q of a token is the same for every column: once a chunk, a warp a token, instead of once a column
-      for (int tc = warp; tc < cn; tc += static_cast<int>(blockDim.x >> 5)) {
+    if (c0 + chunk < n) fetch(c0 + chunk, buffers + (turn ^ 1) * buf_floats);
+    if (MODE != kDeltaPlain) {
+      for (int tc = warp; tc < cn; tc += kDeltaThreads / 32) {
         float dot = 0.0f;
         for (int d = lane; d < dim; d += 32)
-          dot = fmaf(BONUS ? kb[tc * dim + d] * bonus[h * dim + d] : kb[tc * dim + d], qb[tc * dim + d], dot);
+          dot = fmaf(MODE == kDeltaBonus ? kb[tc * dim + d] * bonus[h * dim + d] : kb[tc * dim + d], qb[tc * dim + d], dot);
         dot = warp_sum(dot);
         if (lane == 0) kq[tc] = dot;
       }
       __syncthreads();
     }
-    for (int tc = 0; tc < cn; ++tc) {
+    // One token: this lane's share of the read-out.
+    auto step = [&](int tc) -> float {
       const float* kt = kb + tc * dim;
       const float* qt = qb + tc * dim;
-      const float* gt = gb + tc * dim;
-      float kreg[RMAX];
-      float d1a = 0.0f, d1b = 0.0f, d2a = 0.0f, d2b = 0.0f, d3 = 0.0f;     // d3: k . q over this lane's channels
+      const float* gt = gb + tc * g_ld;
+      const float g1 = decay_per_head ? gt[0] : 1.0f;
+      const float v = vb[tc * kDeltaCols + cidx], be = bb[tc];
+      float kr[R], y0 = 0.0f, y1 = 0.0f, d0 = 0.0f, d1 = 0.0f;
+      float u = be * v;
 #pragma unroll
-      for (int q4 = 0; q4 < RMAX / 4; ++q4) {
-        const int r0 = delta_row<LANES>(4 * q4, lane8);
-        float kk[4], qq[4], gg[4];
-        if (vec4) {                              // dim % 4 == 0: the lane's four channels are one 16-byte piece
+      for (int q4 = 0; q4 < R / 4; ++q4) {
+        const int r0 = delta_row(4 * q4, lane8);
+        float kk[4] = {0.0f, 0.0f, 0.0f, 0.0f}, qq[4] = {0.0f, 0.0f, 0.0f, 0.0f}, gg[4] = {g1, g1, g1, g1};
+        if (vec4) {                              // the lane's four channels are one 16-byte piece
           if (r0 < dim) {
-            const float4 k4 = *reinterpret_cast<const float4*>(kt + r0), q4v = *reinterpret_cast<const float4*>(qt + r0);
-            const float4 g4 = decay_per_head ? make_float4(gt[0], gt[0], gt[0], gt[0]) : *reinterpret_cast<const float4*>(gt + r0);
-            kk[0] = k4.x, kk[1] = k4.y, kk[2] = k4.z, kk[3] = k4.w;
-            qq[0] = q4v.x, qq[1] = q4v.y, qq[2] = q4v.z, qq[3] = q4v.w;
-            gg[0] = g4.x, gg[1] = g4.y, gg[2] = g4.z, gg[3] = g4.w;
-          } else {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) kk[e] = qq[e] = gg[e] = 0.0f;
+            load4(kt + r0, kk);
+            load4(qt + r0, qq);
+            if (!decay_per_head) load4(gt + r0, gg);
           }
         } else {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            const bool in = r0 + e < dim;
-            kk[e] = in ? kt[r0 + e] : 0.0f;
-            qq[e] = in ? qt[r0 + e] : 0.0f;
-            gg[e] = in ? gt[decay_per_head ? 0 : r0 + e] : 0.0f;
+            if (r0 + e < dim) {
+              kk[e] = kt[r0 + e];
+              qq[e] = qt[r0 + e];
+              if (!decay_per_head) gg[e] = gt[r0 + e];
+            }
           }
         }
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float s0 = sreg[4 * q4 + e];
-          const float sv = s0 * gg[e];
-          const float seen = BONUS ? s0 : sv;     // what the read-out sees of the state: before or after the decay
-          sreg[4 * q4 + e] = sv;
-          kreg[4 * q4 + e] = kk[e];
-          if (e & 1) {
-            if (!PLAIN) d1b = fmaf(kk[e], sv, d1b);
-            d2b = fmaf(qq[e], seen, d2b);
+          const int r = 4 * q4 + e;
+          const float before = sreg[r], kept = before * gg[e];
+          if (MODE == kDeltaRule) {
+            sreg[r] = kept;
+            kr[r] = kk[e];
+            if (e & 1) d1 = fmaf(kk[e], kept, d1), y1 = fmaf(qq[e], kept, y1);
+            else d0 = fmaf(kk[e], kept, d0), y0 = fmaf(qq[e], kept, y0);
           } else {
-            if (!PLAIN) d1a = fmaf(kk[e], sv, d1a);
-            d2a = fmaf(qq[e], seen, d2a);
+            sreg[r] = fmaf(kk[e], u, kept);
+            const float seen = MODE == kDeltaBonus ? before : sreg[r];
+            if (e & 1) y1 = fmaf(qq[e], seen, y1);
+            else y0 = fmaf(qq[e], seen, y0);
           }
-          if (!PLAIN) d3 = fmaf(kk[e], qq[e], d3);
         }
       }
-      float d1 = d1a + d1b, d2 = d2a + d2b;
+      float y = y0 + y1;
+      if (MODE == kDeltaRule) {
+        float d = d0 + d1;
 #pragma unroll
-      for (int o = 1; o < LANES; o <<= 1) {
-        if (!PLAIN) d1 += __shfl_xor_sync(0xffffffffu, d1, o);
-        d2 += __shfl_xor_sync(0xffffffffu, d2, o);
-        if (!PLAIN) d3 += __shfl_xor_sync(0xffffffffu, d3, o);
+        for (int o = 1; o < kDeltaLanes; o <<= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
+        u = be * (v - d);
+#pragma unroll
+        for (int r = 0; r < R; ++r) sreg[r] = fmaf(kr[r], u, sreg[r]);
       }
-      const float u = PLAIN ? bb[tc] * vb[tc * kDeltaCols + cidx] : bb[tc] * (vb[tc * kDeltaCols + cidx] - d1);
-      if (PLAIN) d3 = kq[tc];
-      if (live && lane8 == 0) out[(t0 + c0 + tc) * static_cast<long long>(nv) + h * vdim + col] = fmaf(d3, u, d2);
+      if (MODE != kDeltaPlain && lane8 == 0) y = fmaf(kq[tc], u, y);
+      return y;
+    };
+    // Four tokens' shares to sums: lane l of a column ends up with the token l & 3.
+    auto finish = [&](int tb, float (&y)[kDeltaBatch]) {
 #pragma unroll
-      for (int r = 0; r < RMAX; ++r) sreg[r] = fmaf(kreg[r], u, sreg[r]);
+      for (int q = 0; q < 2; ++q) {
+        const bool up = lane8 & 2;
+        const float give = up ? y[q] : y[q + 2], keep = up ? y[q + 2] : y[q];
+        y[q] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+      }
+      const bool up = lane8 & 1;
+      const float give = up ? y[0] : y[1], keep = up ? y[1] : y[0];
+      float sum = keep + __shfl_xor_sync(0xffffffffu, give, 1);
+      sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+      if (live && lane8 < kDeltaBatch && tb + lane8 < cn) out[(t0 + c0 + tb + lane8) * static_cast<long long>(nv) + h * vdim + col] = sum;
+    };
+    int tb = 0;
+    for (; tb + kDeltaBatch <= cn; tb += kDeltaBatch) {
+      float y[kDeltaBatch];
+#pragma unroll
+      for (int q = 0; q < kDeltaBatch; ++q) y[q] = step(tb + q);
+      finish(tb, y);
+    }
+    if (tb < cn) {
+      float y[kDeltaBatch] = {0.0f, 0.0f, 0.0f, 0.0f};
+      for (int q = 0; tb + q < cn; ++q) {
+        const float v = step(tb + q);
+        if (q == 0) y[0] = v;
+        else if (q == 1) y[1] = v;
+        else y[2] = v;
+      }
+      finish(tb, y);
     }
   }
   pdl_launch_dependents();
-  __syncthreads();
 #pragma unroll
-  for (int r = 0; r < RMAX; ++r) {
-    const int rowi = delta_row<LANES>(r, lane8);
-    if (rowi < dim) smem[rowi * kDeltaPad + cidx] = sreg[r];
+  for (int r = 0; r < R; ++r) {
+    const int rowi = delta_row(r, lane8);
+    if (rowi < dim) stage[rowi * kDeltaPad + cidx] = sreg[r];
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < dim * kDeltaCols; i += blockDim.x) {
-    const int r = i / kDeltaCols, c = i % kDeltaCols;
-    if (col0 + c < vdim) S[static_cast<long long>(r) * vdim + col0 + c] = smem[r * kDeltaPad + c];
+  if (quads) {
+#pragma unroll 4
+    for (int i = threadIdx.x; i < dim * (kDeltaCols / 4); i += kDeltaThreads) {
+      const int r = i / (kDeltaCols / 4), c = (i % (kDeltaCols / 4)) * 4;
+      float v[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = stage[r * kDeltaPad + c + e];
+      if (col0 + c < vdim) store4(S + static_cast<long long>(r) * vdim + col0 + c, v);
+    }
+  } else {
+    for (int i = threadIdx.x; i < dim * kDeltaCols; i += kDeltaThreads) {
+      const int r = i / kDeltaCols, c = i % kDeltaCols;
+      if (col0 + c < vdim) S[static_cast<long long>(r) * vdim + col0 + c] = stage[r * kDeltaPad + c];
+    }
   }
   // The convolution's last taps - 1 inputs after this step: from the step's rows where it brought enough, else
   // what the slot held moves up. Every block of the sequence takes a slice of the channels.
@@ -388,44 +444,55 @@ static int launch_delta_rule(const float* qn, const float* kn, const float* vn, 
                              long long decay_stride, float* state, long long state_stride, long long conv_state_off,
                              const void* proj, long long proj_stride, int q_off, int k_off, int v_off,
                              const int* query_start, const int* state_slots, int seqs, const DeltaShape& sh, float* out,
-                             int plain, int decay_per_head, cudaStream_t s, const float* bonus = nullptr) {
+                             int plain, int decay_per_head, int single, cudaStream_t s, const float* bonus = nullptr) {
   const dim3 grid(seqs, sh.heads, ceil_div(sh.vdim, kDeltaCols));
-  const int per_token = 3 * sh.dim + kDeltaCols + 1;
-  int chunk = (44 * 1024 / static_cast<int>(sizeof(float))) / (2 * per_token);      // two buffers
-  chunk = chunk > 16 ? 16 : (chunk < 1 ? 1 : chunk);
-  const int stage = sh.dim * kDeltaPad;                         // the state tile on its way in and out
-  const int buffers = 2 * ((chunk * per_token + 3) & ~3) + 16;        // and a chunk's k . q (the plain mode)
-  const int floats = buffers > stage ? buffers : stage;
+  const int per_token = 2 * sh.dim + (decay_per_head ? 1 : sh.dim) + kDeltaCols + 1;
+  int chunk = kDeltaBatch;                     // `single`: one token a sequence, small buffers, many blocks an SM
+  if (!single) {
+    chunk = (60 * 1024 / static_cast<int>(sizeof(float))) / (2 * per_token) / kDeltaBatch * kDeltaBatch;      // two buffers
+    chunk = chunk > 32 ? 32 : (chunk < kDeltaBatch ? kDeltaBatch : chunk);
+  }
+  const int floats = ((sh.dim * kDeltaPad + 3) & ~3) + 2 * ((chunk * per_token + 3) & ~3) + chunk;
   const size_t smem = static_cast<size_t>(floats) * sizeof(float);
   const T* p = static_cast<const T*>(proj);
-#define TIE_DELTA_CASE(R, LANES)                                                                                          \
-  do {                                                                                                                    \
-    if (plain && bonus)                                                                                                   \
-      tie::launch_kernel_alone(delta_rule_kernel<T, R, LANES, true, true>, grid, dim3(LANES * kDeltaCols), smem, s, qn, kn, vn, beta, decay, \
-                         decay_stride, state, state_stride, conv_state_off, p, proj_stride, q_off, k_off, v_off, query_start,   \
-                         state_slots, sh, chunk, out, decay_per_head, bonus);                                             \
-    else if (plain)                                                                                                       \
-      tie::launch_kernel_alone(delta_rule_kernel<T, R, LANES, true>, grid, dim3(LANES * kDeltaCols), smem, s, qn, kn, vn, beta, decay, \
-                         decay_stride, state, state_stride, conv_state_off, p, proj_stride, q_off, k_off, v_off, query_start,   \
-                         state_slots, sh, chunk, out, decay_per_head, nullptr);                                           \
-    else                                                                                                                  \
-      tie::launch_kernel_alone(delta_rule_kernel<T, R, LANES, false>, grid, dim3(LANES * kDeltaCols), smem, s, qn, kn, vn, beta, decay, \
-                         decay_stride, state, state_stride, conv_state_off, p, proj_stride, q_off, k_off, v_off, query_start,   \
-                         state_slots, sh, chunk, out, decay_per_head, nullptr);                                           \
+  int failed = 0;
+  auto run = [&](auto kernel) {
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess) {
+      failed = 1;
+      return;
+    }
+    if (single)
+      TIE_LAUNCH(kernel, grid, kDeltaThreads, smem, s, qn, kn, vn, beta, decay, decay_stride, state, state_stride, conv_state_off, p,
+                 proj_stride, q_off, k_off, v_off, query_start, state_slots, sh, chunk, out, decay_per_head, bonus);
+    else
+      launch_kernel_alone(kernel, grid, dim3(kDeltaThreads), smem, s, qn, kn, vn, beta, decay, decay_stride, state, state_stride,
+                          conv_state_off, p, proj_stride, q_off, k_off, v_off, query_start, state_slots, sh, chunk, out, decay_per_head,
+                          bonus);
+  };
+#define TIE_DELTA_CASE(R)                                                    \
+  do {                                                                       \
+    if (bonus != nullptr) run(delta_rule_kernel<T, R, kDeltaBonus>);         \
+    else if (plain) run(delta_rule_kernel<T, R, kDeltaPlain>);               \
+    else run(delta_rule_kernel<T, R, kDeltaRule>);                           \
   } while (0)
-  if (sh.dim <= 32) TIE_DELTA_CASE(4, 8);
-  else if (sh.dim <= 64) TIE_DELTA_CASE(4, 16);
-  else if (sh.dim <= 128) TIE_DELTA_CASE(4, 32);
-  else TIE_DELTA_CASE(8, 32);
+  if (sh.dim <= 32) TIE_DELTA_CASE(4);
+  else if (sh.dim <= 64) TIE_DELTA_CASE(8);
+  else if (sh.dim <= 128) TIE_DELTA_CASE(16);
+  else TIE_DELTA_CASE(32);
 #undef TIE_DELTA_CASE
+  if (failed) {
+    set_error("delta_rule: cannot reserve %zu bytes of shared memory", smem);
+    return kCudaError;
+  }
   TIE_RETURN_LAUNCH("delta_rule");
 }
 
+// single != 0: every sequence brings one token.
 TIE_API int tie_delta_rule(int dtype, const float* qn, const float* kn, const float* vn, const float* beta,
                            const float* decay, long long decay_stride, float* state, long long state_stride,
                            long long conv_state_off, const void* proj, long long proj_stride, int q_off, int k_off,
                            int v_off, const int* query_start, const int* state_slots, int seqs, int heads, int kv_heads,
-                           int dim, int vdim, int taps, float* out, int plain, int decay_per_head, cudaStream_t s) {
+                           int dim, int vdim, int taps, float* out, int plain, int decay_per_head, int single, cudaStream_t s) {
   const DeltaShape sh{heads, kv_heads, dim, vdim, taps};
   if (const int st_ = check_delta(sh)) return st_;
   if (seqs <= 0) return kOk;
@@ -433,10 +500,10 @@ TIE_API int tie_delta_rule(int dtype, const float* qn, const float* kn, const fl
   TIE_REQUIRE(seqs <= 65535 * 32 && heads <= 65535, "delta_rule: %d sequences x %d heads exceed the grid", seqs, heads);
   if (dtype == TIE_F32)
     return launch_delta_rule<float>(qn, kn, vn, beta, decay, decay_stride, state, state_stride, conv_state_off, proj, proj_stride,
-                                    q_off, k_off, v_off, query_start, state_slots, seqs, sh, out, plain, decay_per_head, s);
+                                    q_off, k_off, v_off, query_start, state_slots, seqs, sh, out, plain, decay_per_head, single, s);
   if (dtype == TIE_BF16)
     return launch_delta_rule<__nv_bfloat16>(qn, kn, vn, beta, decay, decay_stride, state, state_stride, conv_state_off, proj,
-                                            proj_stride, q_off, k_off, v_off, query_start, state_slots, seqs, sh, out, plain, decay_per_head, s);
+                                            proj_stride, q_off, k_off, v_off, query_start, state_slots, seqs, sh, out, plain, decay_per_head, single, s);
   set_error("unknown dtype code %d", dtype);
   return kBadArgument;
 }
@@ -460,12 +527,12 @@ TIE_API int tie_delta_out(int dtype, const float* o, const float* gate, long lon
 }
 
 // The plain recurrence read before it is written, with a weight per head and key channel on the token's own write
-// (`bonus`, float [heads * dim]): o_t = (S + diag(bonus) k_t u_t^T)^T q_t, then S <- diag(decay_t) S + k_t u_t^T.
+// (`bonus`, float [heads * dim]; `single` as above): o_t = (S + diag(bonus) k_t u_t^T)^T q_t, then S <- diag(decay_t) S + k_t u_t^T.
 TIE_API int tie_delta_rule_bonus(int dtype, const float* qn, const float* kn, const float* vn, const float* beta,
                                  const float* decay, long long decay_stride, float* state, long long state_stride,
                                  long long conv_state_off, const void* proj, long long proj_stride, int q_off, int k_off,
                                  int v_off, const int* query_start, const int* state_slots, int seqs, int heads,
-                                 int kv_heads, int dim, int vdim, int taps, float* out, const float* bonus, cudaStream_t s) {
+                                 int kv_heads, int dim, int vdim, int taps, float* out, const float* bonus, int single, cudaStream_t s) {
   const DeltaShape sh{heads, kv_heads, dim, vdim, taps};
   if (const int st_ = check_delta(sh)) return st_;
   if (seqs <= 0) return kOk;
@@ -473,10 +540,10 @@ TIE_API int tie_delta_rule_bonus(int dtype, const float* qn, const float* kn, co
   TIE_REQUIRE(seqs <= 65535 * 32 && heads <= 65535, "delta_rule: %d sequences x %d heads exceed the grid", seqs, heads);
   if (dtype == TIE_F32)
     return launch_delta_rule<float>(qn, kn, vn, beta, decay, decay_stride, state, state_stride, conv_state_off, proj, proj_stride,
-                                    q_off, k_off, v_off, query_start, state_slots, seqs, sh, out, 1, 0, s, bonus);
+                                    q_off, k_off, v_off, query_start, state_slots, seqs, sh, out, 1, 0, single, s, bonus);
   if (dtype == TIE_BF16)
     return launch_delta_rule<__nv_bfloat16>(qn, kn, vn, beta, decay, decay_stride, state, state_stride, conv_state_off, proj,
-                                            proj_stride, q_off, k_off, v_off, query_start, state_slots, seqs, sh, out, 1, 0, s, bonus);
+                                            proj_stride, q_off, k_off, v_off, query_start, state_slots, seqs, sh, out, 1, 0, single, s, bonus);
   set_error("unknown dtype code %d", dtype);
   return kBadArgument;
 }

@@ -185,20 +185,29 @@ __global__ void __launch_bounds__(LANES * kScanChannels) selective_scan_kernel(S
       cs[i] = p < a.states ? ld(cb + tc * L.n8 + p) : 0.0f;
     }
     __syncthreads();
+    // One token: this lane's share of the read-out.
+    auto step = [&](int tc) -> float {
+      const float2 d = steps[tc * kScanChannels + ch];
+      const float* bt = bs + tc * L.np + lane * R;
+      const float* ct = cs + tc * L.np + lane * R;
+      float y = 0.0f;
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        sr[r] = fmaf(decay_ex2<T>(d.x * ar[r]), sr[r], d.y * bt[r]);
+        y = fmaf(sr[r], ct[r], y);
+      }
+      return y;
+    };
     for (int tb = 0; tb < cn; tb += 8) {
       float y[8];
+      if (tb + 8 <= cn) {                      // no test between the tokens: their loads and exponentials overlap
 #pragma unroll
-      for (int q = 0; q < 8; ++q) {
-        y[q] = 0.0f;
-        if (tb + q < cn) {
-          const float2 d = steps[(tb + q) * kScanChannels + ch];
-          const float* bt = bs + (tb + q) * L.np + lane * R;
-          const float* ct = cs + (tb + q) * L.np + lane * R;
+        for (int q = 0; q < 8; ++q) y[q] = step(tb + q);
+      } else {
 #pragma unroll
-          for (int r = 0; r < R; ++r) {
-            sr[r] = fmaf(decay_ex2<T>(d.x * ar[r]), sr[r], d.y * bt[r]);
-            y[q] = fmaf(sr[r], ct[r], y[q]);
-          }
+        for (int q = 0; q < 8; ++q) {
+          y[q] = 0.0f;
+          if (tb + q < cn) y[q] = step(tb + q);
         }
       }
       // sums over the lanes: after the exchange over 4, 2, 1 lanes a lane holds one token (the one of its three low bits)

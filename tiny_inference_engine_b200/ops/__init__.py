@@ -705,14 +705,14 @@ def delta_prep(proj, q_off: int, k_off: int, v_off: int, b_off: int, conv_w, sta
 
 def delta_rule(qn, kn, vn, beta, decay, state, conv_state_off: int, proj, q_off: int, k_off: int, v_off: int,
                query_start, state_slots, seqs: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, out,
-               plain: bool = False, decay_per_head: bool = False) -> None:
+               plain: bool = False, decay_per_head: bool = False, single: bool = False) -> None:
     """The recurrence over each sequence's tokens of the step: per head S <- decay S; u = beta (v - S^T k);
     S <- S + k u^T; o = S^T q, with `decay` float32 [T, >= heads * dim] per head and key channel (`delta_prep`).
     S [heads, dim, vdim] sits at the start of the sequence's row of `state` and is updated; so are the convolution's
     last inputs (from the q, k, v columns of `proj`). out float32 [T, heads * vdim].
     `plain`: no correction, u = beta v (beta None: u = v), which is the recurrence of gated linear attention and of
     state-space layers, S <- diag(decay) S + k u^T. `decay_per_head`: decay is float32 [T, >= heads], one factor for
-    all key channels of a head."""
+    all key channels of a head. `single`: every sequence brings one token (a hint: how the launch is cut, not what it computes)."""
     _dev(qn, kn, vn, beta, decay, state, proj, query_start, state_slots, out)
     T = proj.shape[0]
     _need(beta is not None or plain, "delta_rule: the delta rule needs beta")
@@ -725,7 +725,7 @@ def delta_rule(qn, kn, vn, beta, decay, state, conv_state_off: int, proj, q_off:
     call("tie_delta_rule", dtype_code(proj), qn.data_ptr(), kn.data_ptr(), vn.data_ptr(), _ptr(beta), decay.data_ptr(),
          decay.stride(0), state.data_ptr(), state.stride(0), conv_state_off, proj.data_ptr(), proj.stride(0), q_off, k_off, v_off,
          query_start.data_ptr(), state_slots.data_ptr(), seqs, heads, kv_heads, dim, vdim, taps, out.data_ptr(),
-         1 if plain else 0, 1 if decay_per_head else 0, _stream())
+         1 if plain else 0, 1 if decay_per_head else 0, 1 if single else 0, _stream())
 
 
 def delta_out(o, gate, weight, eps: float, out, heads: int, vdim: int) -> None:
@@ -1546,7 +1546,7 @@ def delta_rule_bonus(qn, kn, vn, decay, bonus, state, ctx, heads: int, dim: int,
           "delta_rule_bonus: state rows too short")
     call("tie_delta_rule_bonus", F32, qn.data_ptr(), kn.data_ptr(), vn.data_ptr(), 0, decay.data_ptr(), decay.stride(0), state.data_ptr(),
          state.stride(0), heads * dim * dim, qn.data_ptr(), qn.stride(0), 0, 0, 0, ctx.query_start.data_ptr(), ctx.state_slots.data_ptr(),
-         ctx.S, heads, heads, dim, dim, 1, out.data_ptr(), bonus.data_ptr(), _stream())
+         ctx.S, heads, heads, dim, dim, 1, out.data_ptr(), bonus.data_ptr(), 1 if ctx.multi_seqs == 0 else 0, _stream())
 
 
 def time_mix_out(o, gate, weight, eps: float, out, heads: int, dim: int, h, state, prev_off: int, ctx) -> None:

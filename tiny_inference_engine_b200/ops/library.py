@@ -49,7 +49,7 @@ _SIGNATURES = {
     "tie_scale_rows": [P, L, I, I, F, P],
     "tie_qkv_span_prep": [I, P, L, I, I, I, P, P, P, P, P, F, P, I, P, P, P, P, I, I, I, I, I, I, I, I, P, P, P],
     "tie_delta_prep": [I, P, L, I, I, I, I, P, P, L, L, P, P, P, I, I, I, I, I, I, F, F, P, P, P, P, P, L, P, P, P],
-    "tie_delta_rule": [I, P, P, P, P, P, L, P, L, L, P, L, I, I, I, P, P, I, I, I, I, I, I, P, I, I, P],
+    "tie_delta_rule": [I, P, P, P, P, P, L, P, L, L, P, L, I, I, I, P, P, I, I, I, I, I, I, P, I, I, I, P],
     "tie_delta_out": [I, P, P, L, P, F, P, I, I, I, P],
     "tie_gemm_simt_batched": [I, I, P, P, P, I, I, I, L, L, L, I, L, L, L, P],
     "tie_gla_prep": [I, P, L, I, I, I, I, I, I, I, F, F, P, P, P, P, P, L, P],
@@ -82,7 +82,7 @@ _SIGNATURES = {
     "tie_attention_maps_rows": [I, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, I, F, F, P, P, I, P],
     "tie_attention_maps_split": [I, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, P, P, I, P, I, I, I, P, P],
     "tie_attention_prompt_maps": [P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, I, I, I, F, P, P, P],
-    "tie_delta_rule_bonus": [I, P, P, P, P, P, L, P, L, L, P, L, I, I, I, P, P, I, I, I, I, I, I, P, P, P],
+    "tie_delta_rule_bonus": [I, P, P, P, P, P, L, P, L, L, P, L, I, I, I, P, P, I, I, I, I, I, I, P, P, I, P],
     "tie_add_tanh_norm": [I, P, P, P, L, I, F, P, P, L, I, F, P, F, P, P, P, I, I, P],
     "tie_sinusoid_add": [P, P, I, I, F, P],
     "tie_slice_norm_append": [I, P, L, I, I, I, I, I, I, I, P, P, F, P, P, P, I, I, I, I, I, I, P],

@@ -125,7 +125,8 @@ class ChannelGatedDelta(Mixer):
                        self.q_scale, qn, kn, vn, beta, a_raw, self.dt_bias, self.a_log)       # a_raw leaves as the decays
         o = ctx.ws.rows("delta.o", T, self.nv, torch.float32)
         ops.delta_rule(qn, kn, vn, beta, a_raw, state, self.state_floats, proj, self.q_off,
-                       self.k_off, self.v_off, ctx.query_start, ctx.state_slots, ctx.S, H, G, dim, vdim, self.taps, o)
+                       self.k_off, self.v_off, ctx.query_start, ctx.state_slots, ctx.S, H, G, dim, vdim, self.taps, o,
+                       single=ctx.multi_seqs == 0)
         gated = ctx.ws.rows("delta.gated", T, self.nv, self.dtype)
         ops.delta_out(o, gate, self.norm_w, self.eps, gated, H, vdim)
         out = ctx.ws.rows("mixer.out", T, self.hidden, self.dtype)

@@ -102,7 +102,7 @@ class GatedLinearAttention(Mixer):
         ops.gla_prep(proj, self.q_off, self.k_off, self.v_off, H, dim, vdim, self.q_scale, self.tau, self.a2_bias, qn, kn, vn, decay)
         o = ctx.ws.rows("gla.o", T, self.nv, torch.float32)
         ops.delta_rule(qn, kn, vn, None, decay, state, self.state_floats, proj, self.q_off, self.k_off, self.v_off,
-                       ctx.query_start, ctx.state_slots, ctx.S, H, H, dim, vdim, 1, o, plain=True)
+                       ctx.query_start, ctx.state_slots, ctx.S, H, H, dim, vdim, 1, o, plain=True, single=ctx.multi_seqs == 0)
         gated = ctx.ws.rows("gla.gated", T, self.nv, self.dtype)
         ops.head_norm_gate(o, proj[:, self.g_off:self.g_off + self.nv], self.norm_w, self.eps, gated, H, vdim, ops.GATE_SILU)
         out = ctx.ws.rows("mixer.out", T, self.hidden, self.dtype)
@@ -175,7 +175,8 @@ class ConstantDecayAttention(Mixer):
         ops.act_split(proj, self.q_off, self.k_off, self.v_off, qn, kn, vn)
         o = ctx.ws.rows("cda.o", T, self.nv, torch.float32)
         ops.delta_rule(qn, kn, vn, None, self.decay.expand(T, H), state, self.state_floats, proj, self.q_off, self.k_off, self.v_off,
-                       ctx.query_start, ctx.state_slots, ctx.S, H, H, dim, vdim, 1, o, plain=True, decay_per_head=True)
+                       ctx.query_start, ctx.state_slots, ctx.S, H, H, dim, vdim, 1, o, plain=True, decay_per_head=True,
+                       single=ctx.multi_seqs == 0)
         gated = ctx.ws.rows("cda.gated", T, self.nv, self.dtype)
         ops.head_norm_gate(o, proj[:, self.g_off:self.g_off + self.nv], self.norm_w, self.eps, gated, 1, self.nv, ops.GATE_SIGMOID)
         out = ctx.ws.rows("mixer.out", T, self.hidden, self.dtype)

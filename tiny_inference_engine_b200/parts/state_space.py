@@ -107,7 +107,7 @@ class StateSpaceDual(Mixer):
                      cn, bn, xn, dt, decay)
         o = ctx.ws.rows("ssd.o", T, self.inner, torch.float32)
         ops.delta_rule(cn, bn, xn, dt, decay, state, self.state_floats, proj, self.c_off, self.b_off, self.x_off,
-                       ctx.query_start, ctx.state_slots, ctx.S, H, G, N, vdim, self.taps, o, plain=True, decay_per_head=True)
+                       ctx.query_start, ctx.state_slots, ctx.S, H, G, N, vdim, self.taps, o, plain=True, decay_per_head=True, single=ctx.multi_seqs == 0)
         gated = ctx.ws.rows("ssd.gated", T, self.inner, self.dtype)
         ops.ssd_out(o, xn, proj[:, self.z_off:self.z_off + self.inner], self.skip, self.norm_w, self.eps, gated, H, vdim,
                     self.norm_parts)
