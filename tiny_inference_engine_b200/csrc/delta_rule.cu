@@ -103,6 +103,99 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const T* __restrict__ p
   for (int d = threadIdx.x, n = 0; d < width && n < 2; d += blockDim.x, ++n) dst[d] = unit < G ? (vals[n] * inv) * q_scale : vals[n] * inv;
 }
 
+// The same with a warp a unit, four channels a lane and four taps: sizes and sections in whole pieces of four.
+template <typename T>
+__global__ void __launch_bounds__(128) delta_prep_warp_kernel(const T* __restrict__ proj, long long stride, int q_off, int k_off,
+                                                              int v_off, int b_off, const float* __restrict__ conv_w,
+                                                              const float* __restrict__ state, long long state_stride,
+                                                              long long conv_state_off, const int* __restrict__ seq_of_row,
+                                                              const int* __restrict__ query_start,
+                                                              const int* __restrict__ state_slots, DeltaShape sh, float unit_eps,
+                                                              float q_scale, float* __restrict__ qn, float* __restrict__ kn,
+                                                              float* __restrict__ vn, float* __restrict__ beta,
+                                                              float* __restrict__ decay, long long decay_stride,
+                                                              const float* __restrict__ dt_bias, const float* __restrict__ a_log) {
+  pdl_sync();
+  const int t = blockIdx.x, unit = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int G = sh.kv_heads, H = sh.heads, dim = sh.dim, vdim = sh.vdim;
+  const int nqk = G * dim, nv = H * vdim, C = 2 * nqk + nv;
+  if (unit > 2 * G + 2 * H) return;
+  const T* row = proj + static_cast<long long>(t) * stride;
+  if (unit == 2 * G + 2 * H) {
+    for (int h = lane; h < H; h += 32) beta[static_cast<long long>(t) * H + h] = sigmoidf_(ld(row + b_off + h));
+    return;
+  }
+  if (unit >= 2 * G + H) {
+    const int h = unit - (2 * G + H);
+    const float rate = expf(a_log[h]);
+    float* a = decay + static_cast<long long>(t) * decay_stride + h * dim;
+    for (int d = lane * 4; d < dim; d += 128) {
+      float z[4], b[4];
+      load4(a + d, z);
+      load4(dt_bias + h * dim + d, b);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) z[e] = expf(-rate * softplusf_(z[e] + b[e]));
+      store4(a + d, z);
+    }
+    return;
+  }
+  const int s = seq_of_row[t];
+  const int j = t - query_start[s];
+  const int slot = state_slots[s];
+  const float* tail = slot >= 0 ? state + slot * state_stride + conv_state_off : nullptr;
+  const bool is_v = unit >= 2 * G;
+  const int width = is_v ? vdim : dim;
+  const int c0 = is_v ? 2 * nqk + (unit - 2 * G) * vdim : unit * dim;
+  const int col0 = is_v ? v_off + (unit - 2 * G) * vdim : (unit < G ? q_off + unit * dim : k_off + (unit - G) * dim);
+  float* dst = is_v ? vn + static_cast<long long>(t) * nv + (unit - 2 * G) * vdim
+                    : (unit < G ? qn + static_cast<long long>(t) * nqk + unit * dim
+                                : kn + static_cast<long long>(t) * nqk + (unit - G) * dim);
+  float kept[2][4], ss = 0.0f;               // dim <= 256: at most two pieces of a q or k head a lane
+#pragma unroll 2
+  for (int n = 0; n * 128 < width; ++n) {
+    const int d = n * 128 + lane * 4;
+    float y[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+    if (d < width) {
+      float in[4][4], w[4][4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int back = 3 - i;
+        load4(conv_w + (c0 + d + i) * 4, w[i]);      // w[e]: the taps of channel d + e
+        if (back <= j) {
+          load4(row - static_cast<long long>(back) * stride + col0 + d, in[i]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) in[i][e] = tail ? tail[static_cast<long long>(j + i) * C + c0 + d + e] : 0.0f;
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) y[e] = fmaf(w[e][i], in[i][e], y[e]);
+        y[e] = y[e] * sigmoidf_(y[e]);
+        ss = fmaf(y[e], y[e], ss);
+      }
+      if (is_v) store4(dst + d, y);
+    }
+    if (n < 2) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) kept[n & 1][e] = y[e];
+    }
+  }
+  if (is_v) return;
+  ss = warp_sum(ss);
+  const float inv = (1.0f / sqrtf(ss + unit_eps)) * (unit < G ? q_scale : 1.0f);
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    const int d = n * 128 + lane * 4;
+    if (d < width) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) kept[n][e] *= inv;
+      store4(dst + d, kept[n]);
+    }
+  }
+}
+
 __device__ __forceinline__ void async_copy4(float* dst, const float* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))), "l"(src) : "memory");
 }
@@ -112,15 +205,20 @@ __device__ __forceinline__ void async_copy16(float* dst, const float* src) {
 __device__ __forceinline__ void async_copies_done() { asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory"); }
 
 constexpr int kDeltaCols = 16;       // columns of S that a block holds
-constexpr int kDeltaLanes = 8;       // lanes of a warp that share a column
-constexpr int kDeltaThreads = kDeltaCols * kDeltaLanes;
 constexpr int kDeltaPad = kDeltaCols + 1;
 constexpr int kDeltaBatch = 4;       // tokens whose read-outs are summed over the lanes together
 
 // The key channel that register r of lane `lane` (of the eight that share a column) holds: four channels in a row, then the
 // next four 32 channels on, so that a lane reads its k, q and decay entries 16 bytes at a time and the lanes of a column
 // read 128 bytes in a row (the four columns of a warp read the same 128 bytes).
-__device__ __forceinline__ int delta_row(int r, int lane) { return (r >> 2) * (4 * kDeltaLanes) + lane * 4 + (r & 3); }
+template <int LANES>
+__device__ __forceinline__ int delta_row(int r, int lane) { return (r >> 2) * (4 * LANES) + lane * 4 + (r & 3); }
+
+// A token's rows as a lane holds them.
+template <int R, bool ONE_DECAY>
+struct DeltaToken {
+  float k[R], q[R], g[ONE_DECAY ? 1 : R], v, beta, kq;
+};
 
 // What the recurrence does with a token (u is what it writes along its key):
 //   kDeltaRule   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
@@ -136,26 +234,30 @@ enum DeltaMode { kDeltaRule, kDeltaPlain, kDeltaBonus };
 // read-outs of four tokens are summed over the lanes together (each exchange halves the tokens that a lane still holds), and
 // k . q of a token is formed once a chunk, for all columns. In the delta rule the read-out of the updated state is
 // (gS)^T q + (k . q) u, so it does not wait for the update.
-template <typename T, int R, DeltaMode MODE>
-__global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(
+// FULL: the head has exactly LANES * R key channels and its rows come in whole 16-byte pieces, and what the decays are
+// (PER_HEAD: one a token and head) is known too: no tests inside the walk.
+template <typename T, int R, int LANES, DeltaMode MODE, bool FULL, bool PER_HEAD>
+__global__ void __launch_bounds__(kDeltaCols * LANES) delta_rule_kernel(
     const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ vn, const float* __restrict__ beta,
     const float* __restrict__ decay, long long decay_stride, float* __restrict__ state, long long state_stride,
     long long conv_state_off, const T* __restrict__ proj, long long proj_stride, int q_off, int k_off, int v_off,
     const int* __restrict__ query_start, const int* __restrict__ state_slots, DeltaShape sh, int chunk,
-    float* __restrict__ out, int decay_per_head, const float* __restrict__ bonus = nullptr) {
+    float* __restrict__ out, int decay_per_head_, const float* __restrict__ bonus = nullptr) {
+  const bool decay_per_head = FULL ? PER_HEAD : decay_per_head_ != 0;
   // A block is one long chain of dependent steps, and there are few blocks (sequences x heads x column tiles). Started early
   // (programmatic dependent launch), beside a kernel that still fills the GPU, the blocks were placed on the few SMs that had
   // room first and shared them. So for steps with portions the launcher starts this kernel only when the kernels ahead have
   // drained (launch_kernel_alone), and the kernel behind is let in when the walk over the tokens is done.
   pdl_wait();
+  constexpr int kDeltaThreads = kDeltaCols * LANES;
   extern __shared__ float smem[];
   const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * kDeltaCols;
   const int slot = state_slots[s];
   if (slot < 0) return;                       // a sequence that pads a captured batch
   const int t0 = query_start[s], n = query_start[s + 1] - t0;
-  const int dim = sh.dim, vdim = sh.vdim, nqk = sh.kv_heads * dim, nv = sh.heads * vdim;
+  const int dim = FULL ? LANES * R : sh.dim, vdim = sh.vdim, nqk = sh.kv_heads * dim, nv = sh.heads * vdim;
   const int g = h / (sh.heads / sh.kv_heads);
-  const int lane8 = threadIdx.x % kDeltaLanes, cidx = threadIdx.x / kDeltaLanes, col = col0 + cidx;
+  const int lane8 = threadIdx.x % LANES, cidx = threadIdx.x / LANES, col = col0 + cidx;
   const bool live = col < vdim;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* S = state + slot * state_stride + static_cast<long long>(h) * dim * vdim;
@@ -182,7 +284,7 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(
   const int g_ld = decay_per_head ? 1 : dim;
   const int buf_floats = (chunk * (2 * dim + g_ld + kDeltaCols + 1) + 3) & ~3;      // a buffer starts on a 16-byte boundary
   float* const kq = buffers + 2 * buf_floats;                                       // [chunk]: k . q of the chunk's tokens
-  const bool vec4 = dim % 4 == 0;
+  const bool vec4 = FULL || dim % 4 == 0;
   const bool wide = vec4 && nqk % 4 == 0 && ((reinterpret_cast<uintptr_t>(kn) | reinterpret_cast<uintptr_t>(qn)) & 15) == 0 &&
                     (decay_per_head || (decay_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(decay) & 15) == 0));
   auto fetch = [&](int c0, float* base) {
@@ -226,8 +328,8 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(
   float sreg[R];
 #pragma unroll
   for (int r = 0; r < R; ++r) {
-    const int rowi = delta_row(r, lane8);
-    sreg[r] = rowi < dim ? stage[rowi * kDeltaPad + cidx] : 0.0f;
+    const int rowi = delta_row<LANES>(r, lane8);
+    sreg[r] = FULL || rowi < dim ? stage[rowi * kDeltaPad + cidx] : 0.0f;
   }
   int turn = 0;
   for (int c0 = 0; c0 < n; c0 += chunk, turn ^= 1) {
@@ -250,21 +352,22 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(
       }
       __syncthreads();
     }
-    // One token: this lane's share of the read-out.
-    auto step = [&](int tc) -> float {
+    // What a lane needs of a token. The next token's is fetched from shared memory ahead of this token's exchanges: the chain
+    // from token to token then waits for no load.
+    auto fetch_token = [&](int tc, DeltaToken<R, FULL && PER_HEAD>& x) {
       const float* kt = kb + tc * dim;
       const float* qt = qb + tc * dim;
       const float* gt = gb + tc * g_ld;
+      x.v = vb[tc * kDeltaCols + cidx], x.beta = bb[tc];
+      if (MODE != kDeltaPlain) x.kq = kq[tc];
       const float g1 = decay_per_head ? gt[0] : 1.0f;
-      const float v = vb[tc * kDeltaCols + cidx], be = bb[tc];
-      float kr[R], y0 = 0.0f, y1 = 0.0f, d0 = 0.0f, d1 = 0.0f;
-      float u = be * v;
+      if (FULL && PER_HEAD) x.g[0] = g1;
 #pragma unroll
       for (int q4 = 0; q4 < R / 4; ++q4) {
-        const int r0 = delta_row(4 * q4, lane8);
+        const int r0 = delta_row<LANES>(4 * q4, lane8);
         float kk[4] = {0.0f, 0.0f, 0.0f, 0.0f}, qq[4] = {0.0f, 0.0f, 0.0f, 0.0f}, gg[4] = {g1, g1, g1, g1};
         if (vec4) {                              // the lane's four channels are one 16-byte piece
-          if (r0 < dim) {
+          if (FULL || r0 < dim) {
             load4(kt + r0, kk);
             load4(qt + r0, qq);
             if (!decay_per_head) load4(gt + r0, gg);
@@ -281,31 +384,43 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(
         }
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int r = 4 * q4 + e;
-          const float before = sreg[r], kept = before * gg[e];
-          if (MODE == kDeltaRule) {
-            sreg[r] = kept;
-            kr[r] = kk[e];
-            if (e & 1) d1 = fmaf(kk[e], kept, d1), y1 = fmaf(qq[e], kept, y1);
-            else d0 = fmaf(kk[e], kept, d0), y0 = fmaf(qq[e], kept, y0);
-          } else {
-            sreg[r] = fmaf(kk[e], u, kept);
-            const float seen = MODE == kDeltaBonus ? before : sreg[r];
-            if (e & 1) y1 = fmaf(qq[e], seen, y1);
-            else y0 = fmaf(qq[e], seen, y0);
-          }
+          x.k[4 * q4 + e] = kk[e], x.q[4 * q4 + e] = qq[e];
+          if (!(FULL && PER_HEAD)) x.g[4 * q4 + e] = gg[e];
+        }
+      }
+    };
+    DeltaToken<R, FULL && PER_HEAD> ahead;
+    fetch_token(0, ahead);
+    // One token: this lane's share of the read-out.
+    auto step = [&](int tc) -> float {
+      const DeltaToken<R, FULL && PER_HEAD> x = ahead;
+      fetch_token(min(tc + 1, cn - 1), ahead);
+      float y0 = 0.0f, y1 = 0.0f, d0 = 0.0f, d1 = 0.0f;
+      float u = x.beta * x.v;
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        const float before = sreg[r], kept = before * x.g[FULL && PER_HEAD ? 0 : r];
+        if (MODE == kDeltaRule) {
+          sreg[r] = kept;
+          if (r & 1) d1 = fmaf(x.k[r], kept, d1), y1 = fmaf(x.q[r], kept, y1);
+          else d0 = fmaf(x.k[r], kept, d0), y0 = fmaf(x.q[r], kept, y0);
+        } else {
+          sreg[r] = fmaf(x.k[r], u, kept);
+          const float seen = MODE == kDeltaBonus ? before : sreg[r];
+          if (r & 1) y1 = fmaf(x.q[r], seen, y1);
+          else y0 = fmaf(x.q[r], seen, y0);
         }
       }
       float y = y0 + y1;
       if (MODE == kDeltaRule) {
         float d = d0 + d1;
 #pragma unroll
-        for (int o = 1; o < kDeltaLanes; o <<= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-        u = be * (v - d);
+        for (int o = 1; o < LANES; o <<= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
+        u = x.beta * (x.v - d);
 #pragma unroll
-        for (int r = 0; r < R; ++r) sreg[r] = fmaf(kr[r], u, sreg[r]);
+        for (int r = 0; r < R; ++r) sreg[r] = fmaf(x.k[r], u, sreg[r]);
       }
-      if (MODE != kDeltaPlain && lane8 == 0) y = fmaf(kq[tc], u, y);
+      if (MODE != kDeltaPlain && lane8 == 0) y = fmaf(x.kq, u, y);
       return y;
     };
     // Four tokens' shares to sums: lane l of a column ends up with the token l & 3.
@@ -319,7 +434,8 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(
       const bool up = lane8 & 1;
       const float give = up ? y[0] : y[1], keep = up ? y[1] : y[0];
       float sum = keep + __shfl_xor_sync(0xffffffffu, give, 1);
-      sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+#pragma unroll
+      for (int o = 4; o < LANES; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
       if (live && lane8 < kDeltaBatch && tb + lane8 < cn) out[(t0 + c0 + tb + lane8) * static_cast<long long>(nv) + h * vdim + col] = sum;
     };
     int tb = 0;
@@ -343,7 +459,7 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_rule_kernel(
   pdl_launch_dependents();
 #pragma unroll
   for (int r = 0; r < R; ++r) {
-    const int rowi = delta_row(r, lane8);
+    const int rowi = delta_row<LANES>(r, lane8);
     if (rowi < dim) stage[rowi * kDeltaPad + cidx] = sreg[r];
   }
   __syncthreads();
@@ -424,6 +540,21 @@ TIE_API int tie_delta_prep(int dtype, const void* proj, long long stride, int q_
   const int units = 2 * kv_heads + 2 * heads + 1;
   TIE_REQUIRE(units <= 65535, "delta_prep: %d heads exceed the grid", heads);
   const dim3 grid(tokens, units);
+  auto on16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (taps == 4 && dim % 4 == 0 && vdim % 4 == 0 && stride % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && v_off % 4 == 0 &&
+      decay_stride % 4 == 0 && on16(proj) && on16(conv_w) && on16(qn) && on16(kn) && on16(vn) && on16(decay) && on16(dt_bias) &&
+      (dtype == TIE_F32 || dtype == TIE_BF16)) {
+    const dim3 warps(tokens, ceil_div(units, 4));
+    if (dtype == TIE_F32)
+      TIE_LAUNCH((delta_prep_warp_kernel<float>), warps, 128, 0, s, static_cast<const float*>(proj), stride, q_off, k_off, v_off, b_off,
+                 conv_w, state, state_stride, conv_state_off, seq_of_row, query_start, state_slots, sh, unit_eps, q_scale, qn, kn, vn,
+                 beta, decay, decay_stride, dt_bias, a_log);
+    else
+      TIE_LAUNCH((delta_prep_warp_kernel<__nv_bfloat16>), warps, 128, 0, s, static_cast<const __nv_bfloat16*>(proj), stride, q_off, k_off,
+                 v_off, b_off, conv_w, state, state_stride, conv_state_off, seq_of_row, query_start, state_slots, sh, unit_eps, q_scale,
+                 qn, kn, vn, beta, decay, decay_stride, dt_bias, a_log);
+    TIE_RETURN_LAUNCH("delta_prep");
+  }
   if (dtype == TIE_F32) {
     TIE_LAUNCH((delta_prep_kernel<float>), grid, 128, 0, s, static_cast<const float*>(proj), stride, q_off, k_off, v_off, b_off,
                conv_w, state, state_stride, conv_state_off, seq_of_row, query_start, state_slots, sh, unit_eps, q_scale, qn, kn,
@@ -456,29 +587,39 @@ static int launch_delta_rule(const float* qn, const float* kn, const float* vn, 
   const size_t smem = static_cast<size_t>(floats) * sizeof(float);
   const T* p = static_cast<const T*>(proj);
   int failed = 0;
+  const int threads = kDeltaCols * (sh.dim <= 32 ? 8 : 16);
   auto run = [&](auto kernel) {
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess) {
       failed = 1;
       return;
     }
     if (single)
-      TIE_LAUNCH(kernel, grid, kDeltaThreads, smem, s, qn, kn, vn, beta, decay, decay_stride, state, state_stride, conv_state_off, p,
+      TIE_LAUNCH(kernel, grid, threads, smem, s, qn, kn, vn, beta, decay, decay_stride, state, state_stride, conv_state_off, p,
                  proj_stride, q_off, k_off, v_off, query_start, state_slots, sh, chunk, out, decay_per_head, bonus);
     else
-      launch_kernel_alone(kernel, grid, dim3(kDeltaThreads), smem, s, qn, kn, vn, beta, decay, decay_stride, state, state_stride,
+      launch_kernel_alone(kernel, grid, dim3(threads), smem, s, qn, kn, vn, beta, decay, decay_stride, state, state_stride,
                           conv_state_off, p, proj_stride, q_off, k_off, v_off, query_start, state_slots, sh, chunk, out, decay_per_head,
                           bonus);
   };
-#define TIE_DELTA_CASE(R)                                                    \
-  do {                                                                       \
-    if (bonus != nullptr) run(delta_rule_kernel<T, R, kDeltaBonus>);         \
-    else if (plain) run(delta_rule_kernel<T, R, kDeltaPlain>);               \
-    else run(delta_rule_kernel<T, R, kDeltaRule>);                           \
+#define TIE_DELTA_CASE(R, LANES)                                                                    \
+  do {                                                                                       \
+    const bool full = sh.dim == LANES * R;                                             \
+    if (bonus != nullptr) {                                                                  \
+      if (full) run(delta_rule_kernel<T, R, LANES, kDeltaBonus, true, false>);                      \
+      else run(delta_rule_kernel<T, R, LANES, kDeltaBonus, false, false>);                          \
+    } else if (plain) {                                                                      \
+      if (full && decay_per_head) run(delta_rule_kernel<T, R, LANES, kDeltaPlain, true, true>);     \
+      else if (full) run(delta_rule_kernel<T, R, LANES, kDeltaPlain, true, false>);                 \
+      else run(delta_rule_kernel<T, R, LANES, kDeltaPlain, false, false>);                          \
+    } else {                                                                                 \
+      if (full && !decay_per_head) run(delta_rule_kernel<T, R, LANES, kDeltaRule, true, false>);    \
+      else run(delta_rule_kernel<T, R, LANES, kDeltaRule, false, false>);                           \
+    }                                                                                        \
   } while (0)
-  if (sh.dim <= 32) TIE_DELTA_CASE(4);
-  else if (sh.dim <= 64) TIE_DELTA_CASE(8);
-  else if (sh.dim <= 128) TIE_DELTA_CASE(16);
-  else TIE_DELTA_CASE(32);
+  if (sh.dim <= 32) TIE_DELTA_CASE(4, 8);
+  else if (sh.dim <= 64) TIE_DELTA_CASE(4, 16);
+  else if (sh.dim <= 128) TIE_DELTA_CASE(8, 16);
+  else TIE_DELTA_CASE(16, 16);
 #undef TIE_DELTA_CASE
   if (failed) {
     set_error("delta_rule: cannot reserve %zu bytes of shared memory", smem);

@@ -100,6 +100,24 @@ __global__ void __launch_bounds__(256) stream_add_kernel(float* __restrict__ x, 
   }
 }
 
+template <typename T>
+__global__ void __launch_bounds__(256) stream_add_vec4_kernel(float* __restrict__ x, Terms terms, const float* __restrict__ other,
+                                                              const float* __restrict__ vec, long long total4, int D) {
+  pdl_sync();
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total4;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long at = i * 4;
+    float v[4], o[4] = {0.0f, 0.0f, 0.0f, 0.0f}, w[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+    load4(x + at, v);
+    if (other != nullptr) load4(other + at, o);
+    if (vec != nullptr) load4(vec + at % D, w);
+    for (int k = 0; k < terms.n; ++k) term_add4<T>(terms.t[k], at, v);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = (v[e] + o[e]) + w[e];
+    store4(x + at, v);
+  }
+}
+
 }  // namespace tie
 
 using namespace tie;
@@ -161,6 +179,14 @@ TIE_API int tie_stream_add(int dtype, float* x, TIE_TERMS, const float* other, c
   const Terms terms = pack_terms(t0, p0, s0, z0, c0, t1, p1, s1, z1, c1, t2, p2, s2, z2, c2, t3, p3, s3, z3, c3);
   const long long total = static_cast<long long>(n) * D;
   const int blocks = static_cast<int>(min(static_cast<long long>(148 * 8), (total + 255) / 256));
+  auto on16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (D % 4 == 0 && on16(x) && on16(other) && on16(vec) && terms_on16(terms) && (dtype == TIE_F32 || dtype == TIE_BF16)) {
+    const int threads = total / 4 < 148 * 256 ? 64 : 256;      // few rows: spread them over the SMs
+    const int blocks4 = static_cast<int>(min(static_cast<long long>(148 * 8), (total / 4 + threads - 1) / threads));
+    if (dtype == TIE_F32) TIE_LAUNCH((stream_add_vec4_kernel<float>), blocks4, threads, 0, s, x, terms, other, vec, total / 4, D);
+    else TIE_LAUNCH((stream_add_vec4_kernel<__nv_bfloat16>), blocks4, threads, 0, s, x, terms, other, vec, total / 4, D);
+    TIE_RETURN_LAUNCH("stream_add");
+  }
   if (dtype == TIE_F32) {
     TIE_LAUNCH((stream_add_kernel<float>), blocks, 256, 0, s, x, terms, other, vec, total, D);
   } else if (dtype == TIE_BF16) {

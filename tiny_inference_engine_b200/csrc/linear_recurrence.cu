@@ -186,6 +186,40 @@ __global__ void __launch_bounds__(256) head_norm_gate_block_kernel(const float* 
   }
 }
 
+// Four columns a thread, the row in registers between its sum and its use (vdim a multiple of four, at most 4 NV threads).
+template <typename T, int NV>
+__global__ void __launch_bounds__(1024) head_norm_gate_vec4_kernel(const float* __restrict__ o, const T* __restrict__ gate,
+                                                                   long long gate_stride, const float* __restrict__ w, float eps,
+                                                                   T* __restrict__ out, int heads, int vdim, int act) {
+  pdl_sync();
+  __shared__ float scratch[33];
+  const long long item = blockIdx.x, t = item / heads;
+  const int h = static_cast<int>(item % heads);
+  float x[NV][4], gv[NV][4], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = (threadIdx.x + i * blockDim.x) * 4;
+    if (d < vdim) {
+      load4(o + item * vdim + d, x[i]);
+      load4(gate + t * gate_stride + static_cast<long long>(h) * vdim + d, gv[i]);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss = fmaf(x[i][e], x[i][e], ss);
+    }
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(vdim) + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = (threadIdx.x + i * blockDim.x) * 4;
+    if (d < vdim) {
+      float ww[4], r[4];
+      load4(w + d, ww);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) r[e] = ((x[i][e] * inv) * ww[e]) * (act == 1 ? gv[i][e] * lr_sigmoid(gv[i][e]) : lr_sigmoid(gv[i][e]));
+      store4(out + item * vdim + d, r);
+    }
+  }
+}
+
 // y = (o + skip[h] x) * silu(z), each of `parts` equal parts of the row divided by its own root mean square, times w.
 template <typename T>
 __global__ void __launch_bounds__(256) ssd_out_kernel(const float* __restrict__ o, const float* __restrict__ xn,
@@ -285,6 +319,17 @@ TIE_API int tie_head_norm_gate(int dtype, const float* o, const void* gate, long
               tokens, heads, vdim, act);
   const long long items = static_cast<long long>(tokens) * heads;
   if (items == 0) return kOk;
+  auto on16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (vdim >= 512 && vdim % 4 == 0 && vdim <= 8192 && gate_stride % 4 == 0 && items <= 0x7fffffffLL && on16(o) && on16(w) && on16(out) &&
+      reinterpret_cast<uintptr_t>(gate) % 16 == 0) {
+    const int pieces = vdim / 4;
+    int threads = items <= 512 ? 1024 : 256;
+    while (threads < 1024 && pieces > 2 * threads) threads *= 2;
+    while (threads > 32 && threads / 2 >= pieces) threads /= 2;
+    TIE_BY_DTYPE(dtype, TIE_LAUNCH((head_norm_gate_vec4_kernel<T, 2>), static_cast<int>(items), threads, 0, s, o, static_cast<const T*>(gate),
+                                   gate_stride, w, eps, static_cast<T*>(out), heads, vdim, act));
+    TIE_RETURN_LAUNCH("head_norm_gate");
+  }
   if (vdim >= 512 && items <= 0x7fffffffLL) {
     TIE_BY_DTYPE(dtype, TIE_LAUNCH((head_norm_gate_block_kernel<T>), static_cast<int>(items), 256, 0, s, o, static_cast<const T*>(gate),
                                    gate_stride, w, eps, static_cast<T*>(out), heads, vdim, act));

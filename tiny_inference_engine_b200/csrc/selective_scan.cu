@@ -268,8 +268,8 @@ static int launch_scan(ScanArgs<T> a, int seqs, int alone, cudaStream_t s) {
 template <typename T>
 static int scan_of(const ScanArgs<T>& a, int seqs, int alone, cudaStream_t s) {
   if (a.states <= 8) return launch_scan<T, 8, 1>(a, seqs, alone, s);
-  if (a.states <= 16) return launch_scan<T, 8, 2>(a, seqs, alone, s);
-  if (a.states <= 32) return launch_scan<T, 8, 4>(a, seqs, alone, s);
+  if (a.states <= 16) return launch_scan<T, 16, 1>(a, seqs, alone, s);
+  if (a.states <= 32) return launch_scan<T, 16, 2>(a, seqs, alone, s);
   if (a.states <= 64) return launch_scan<T, 16, 4>(a, seqs, alone, s);
   if (a.states <= 128) return launch_scan<T, 32, 4>(a, seqs, alone, s);
   return launch_scan<T, 32, 8>(a, seqs, alone, s);

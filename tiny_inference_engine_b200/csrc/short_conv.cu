@@ -37,6 +37,7 @@ struct ConvArgs {
 };
 
 constexpr int kConvThreads = 128;
+constexpr int kConvMaxTile = 8;
 
 // V channels of a row. VEC: one 16-byte read; else the first n of them one by one.
 template <typename T, int V, bool VEC>
@@ -68,11 +69,26 @@ __device__ __forceinline__ void conv_walk(const ConvArgs& a, int c, int n, int r
     post[e] = a.post != nullptr && e < n ? a.post[c + e] : 0.0f;
   }
   const T* col = static_cast<const T*>(a.proj) + a.col0 + c;
+  // the tile's rows and their sequences, all asked for at once
+  float rows[VEC ? 1 : kConvMaxTile][V];
+  Vec16<T> raw[VEC ? kConvMaxTile : 1];
+  int seqs[kConvMaxTile];
+#pragma unroll
+  for (int i = 0; i < kConvMaxTile; ++i) {
+    if (row0 + i < row1) {
+      seqs[i] = a.seq_of_row[row0 + i];
+      if constexpr (VEC) raw[i].load(col + static_cast<long long>(row0 + i) * a.stride);
+      else conv_load<T, V, VEC>(col + static_cast<long long>(row0 + i) * a.stride, n, rows[i]);
+    }
+  }
   int seq = -1, last = -1;
   bool keeps = false;
   float* tail = nullptr;
-  for (int t = row0; t < row1; ++t) {
-    const int s = a.seq_of_row[t];
+#pragma unroll
+  for (int i8 = 0; i8 < kConvMaxTile; ++i8) {
+    const int t = row0 + i8;
+    if (t >= row1) break;
+    const int s = seqs[i8];
     if (s != seq) {
       seq = s;
       const int q0 = a.query_start[s], q1 = a.query_start[s + 1], slot = a.state_slots[s], j = t - q0;
@@ -97,11 +113,11 @@ __device__ __forceinline__ void conv_walk(const ConvArgs& a, int c, int n, int r
         }
       }
     }
-    conv_load<T, V, VEC>(col + static_cast<long long>(t) * a.stride, n, win[TAPS - 1]);
     float y[V];
 #pragma unroll
     for (int e = 0; e < V; ++e) {
-      win[TAPS - 1][e] += pre[e];
+      if constexpr (VEC) win[TAPS - 1][e] = raw[i8].v[e] + pre[e];
+      else win[TAPS - 1][e] = rows[i8][e] + pre[e];
       y[e] = post[e];
 #pragma unroll
       for (int i = 0; i < TAPS; ++i) y[e] = fmaf(w[i][e], win[i][e], y[e]);
@@ -236,8 +252,8 @@ __global__ void __launch_bounds__(256) conv_tail_kernel(ConvArgs a) {
 using namespace tie;
 
 static int check_conv(const ConvArgs& a, const char* what) {
-  TIE_REQUIRE(a.channels > 0 && a.taps >= 1 && a.taps <= 16 && a.rows >= 0 && a.tile >= 1 && a.w != nullptr,
-              "%s: bad sizes channels=%d taps=%d (1 to 16) rows=%d tile=%d", what, a.channels, a.taps, a.rows, a.tile);
+  TIE_REQUIRE(a.channels > 0 && a.taps >= 1 && a.taps <= 16 && a.rows >= 0 && a.tile >= 1 && a.tile <= kConvMaxTile && a.w != nullptr,
+              "%s: bad sizes channels=%d taps=%d (1 to 16) rows=%d tile=%d (1 to 8)", what, a.channels, a.taps, a.rows, a.tile);
   TIE_REQUIRE(a.taps == 1 || a.state != nullptr, "%s: a convolution of %d taps needs a state", what, a.taps);
   TIE_REQUIRE(ceil_div(a.rows, a.tile) <= 65535, "%s: %d rows in tiles of %d exceed the grid", what, a.rows, a.tile);
   return kOk;
