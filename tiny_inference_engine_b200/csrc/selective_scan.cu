@@ -86,24 +86,27 @@ struct ScanLayout {
 
 template <typename T, int LANES, int R>
 __global__ void __launch_bounds__(LANES * kScanChannels) selective_scan_kernel(ScanArgs<T> a) {
-  pdl_wait();
   extern __shared__ __align__(16) uint8_t scan_smem[];
   constexpr int THREADS = LANES * kScanChannels;
   const int s = blockIdx.y, c0 = blockIdx.x * kScanChannels;
+  const int lane = threadIdx.x % LANES, ch = threadIdx.x / LANES, c = c0 + ch;
+  const bool live = c < a.inner;
+  float sr[R], ar[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {                // a weight: no kernel ahead writes it
+    const int k = lane * R + r;
+    ar[r] = live && k < a.states ? a.a2[static_cast<long long>(c) * a.states + k] : 0.0f;
+  }
+  pdl_wait();
   const int slot = a.state_slots[s];
   if (slot < 0) return;                        // a sequence that pads a captured batch
   const int t0 = a.query_start[s], n = a.query_start[s + 1] - t0;
   const ScanLayout<T> L(a.chunk, a.states, LANES * R);
-  const int lane = threadIdx.x % LANES, ch = threadIdx.x / LANES, c = c0 + ch;
-  const bool live = c < a.inner;
   float* S = a.state + slot * a.state_stride + static_cast<long long>(c) * a.states;
-  float sr[R], ar[R];
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     const int k = lane * R + r;
-    const bool in = live && k < a.states;
-    sr[r] = in ? S[k] : 0.0f;
-    ar[r] = in ? a.a2[static_cast<long long>(c) * a.states + k] : 0.0f;
+    sr[r] = live && k < a.states ? S[k] : 0.0f;
   }
   constexpr int V = Vec16<T>::N;
   auto fetch = [&](int k0, uint8_t* base) {
@@ -251,7 +254,7 @@ __global__ void __launch_bounds__(LANES * kScanChannels) selective_scan_kernel(S
 
 template <typename T, int LANES, int R>
 static int launch_scan(ScanArgs<T> a, int seqs, int alone, cudaStream_t s) {
-  a.chunk = 32;
+  a.chunk = alone ? 32 : 8;                    // single rows: small buffers, many blocks an SM
   while (a.chunk > 8 && ScanLayout<T>(a.chunk, a.states, LANES * R).total > 48 * 1024) a.chunk -= 8;
   const size_t smem = ScanLayout<T>(a.chunk, a.states, LANES * R).total;
   auto kernel = selective_scan_kernel<T, LANES, R>;
@@ -267,6 +270,7 @@ static int launch_scan(ScanArgs<T> a, int seqs, int alone, cudaStream_t s) {
 
 template <typename T>
 static int scan_of(const ScanArgs<T>& a, int seqs, int alone, cudaStream_t s) {
+  if (!alone && a.states <= 16 && a.states > 8) return launch_scan<T, 8, 2>(a, seqs, alone, s);      // single rows: fewer, wider lanes
   if (a.states <= 8) return launch_scan<T, 8, 1>(a, seqs, alone, s);
   if (a.states <= 16) return launch_scan<T, 16, 1>(a, seqs, alone, s);
   if (a.states <= 32) return launch_scan<T, 16, 2>(a, seqs, alone, s);

@@ -39,14 +39,12 @@ struct ConvArgs {
 constexpr int kConvThreads = 128;
 constexpr int kConvMaxTile = 8;
 
-// V channels of a row. VEC: one 16-byte read; else the first n of them one by one.
+// V channels of a row. VEC: four in one read; else the first n of them one by one.
 template <typename T, int V, bool VEC>
 __device__ __forceinline__ void conv_load(const T* p, int n, float (&v)[V]) {
   if constexpr (VEC) {
-    Vec16<T> t;
-    t.load(p);
-#pragma unroll
-    for (int e = 0; e < V; ++e) v[e] = t.v[e];
+    static_assert(V == 4, "rows come four channels at a time");
+    load4(p, v);
   } else {
 #pragma unroll
     for (int e = 0; e < V; ++e) v[e] = e < n ? ld(p + e) : 0.0f;
@@ -70,15 +68,13 @@ __device__ __forceinline__ void conv_walk(const ConvArgs& a, int c, int n, int r
   }
   const T* col = static_cast<const T*>(a.proj) + a.col0 + c;
   // the tile's rows and their sequences, all asked for at once
-  float rows[VEC ? 1 : kConvMaxTile][V];
-  Vec16<T> raw[VEC ? kConvMaxTile : 1];
+  float rows[kConvMaxTile][V];
   int seqs[kConvMaxTile];
 #pragma unroll
   for (int i = 0; i < kConvMaxTile; ++i) {
     if (row0 + i < row1) {
       seqs[i] = a.seq_of_row[row0 + i];
-      if constexpr (VEC) raw[i].load(col + static_cast<long long>(row0 + i) * a.stride);
-      else conv_load<T, V, VEC>(col + static_cast<long long>(row0 + i) * a.stride, n, rows[i]);
+      conv_load<T, V, VEC>(col + static_cast<long long>(row0 + i) * a.stride, n, rows[i]);
     }
   }
   int seq = -1, last = -1;
@@ -116,8 +112,7 @@ __device__ __forceinline__ void conv_walk(const ConvArgs& a, int c, int n, int r
     float y[V];
 #pragma unroll
     for (int e = 0; e < V; ++e) {
-      if constexpr (VEC) win[TAPS - 1][e] = raw[i8].v[e] + pre[e];
-      else win[TAPS - 1][e] = rows[i8][e] + pre[e];
+      win[TAPS - 1][e] = rows[i8][e] + pre[e];
       y[e] = post[e];
 #pragma unroll
       for (int i = 0; i < TAPS; ++i) y[e] = fmaf(w[i][e], win[i][e], y[e]);
@@ -154,10 +149,7 @@ __global__ void __launch_bounds__(kConvThreads) short_conv_act_kernel(ConvArgs a
     }
     T* o = out + t * out_stride + c;
     if constexpr (VEC) {
-      Vec16<T> v;
-#pragma unroll
-      for (int e = 0; e < V; ++e) v.v[e] = y[e];
-      v.store(o);
+      store4(o, y);
     } else {
 #pragma unroll
       for (int e = 0; e < V; ++e)
@@ -189,10 +181,7 @@ __global__ void __launch_bounds__(kConvThreads) conv_rope_append_kernel(ConvArgs
   const int n = min(V, r.dim - d0), row0 = blockIdx.y * a.tile;
   auto put = [&](T* o, const float (&y)[V]) {
     if constexpr (VEC) {
-      Vec16<T> v;
-#pragma unroll
-      for (int e = 0; e < V; ++e) v.v[e] = y[e];
-      v.store(o);
+      store4(o, y);
     } else {
 #pragma unroll
       for (int e = 0; e < V; ++e)
@@ -261,7 +250,7 @@ static int check_conv(const ConvArgs& a, const char* what) {
 
 template <typename T>
 static bool conv_vec(const ConvArgs& a) {
-  constexpr int V = Vec16<T>::N;
+  constexpr int V = 4;
   return a.taps <= 4 && a.stride % V == 0 && a.col0 % V == 0 && reinterpret_cast<uintptr_t>(a.proj) % 16 == 0;
 }
 
@@ -274,7 +263,7 @@ TIE_API int tie_short_conv_act(int dtype, const void* proj, long long stride, in
   if (rows == 0) return kOk;
   auto run = [&](auto* typed) {
     using T = std::remove_pointer_t<decltype(typed)>;
-    constexpr int V = Vec16<T>::N;
+    constexpr int V = 4;
     if (conv_vec<T>(a) && channels % V == 0 && out_stride % V == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0)
       TIE_LAUNCH((short_conv_act_kernel<T, V, 4, true>), dim3(ceil_div(channels / V, kConvThreads), ceil_div(rows, tile)), kConvThreads, 0, s,
                  a, silu, static_cast<T*>(out), out_stride);
@@ -306,7 +295,7 @@ TIE_API int tie_conv_rope_append(int dtype, const void* proj, long long stride, 
   const ConvRopeArgs r{positions, turns, rot, slots, k_cache, v_cache, q_out, q_heads, kv_heads, dim, page_size, k_col};
   auto run = [&](auto* typed) {
     using T = std::remove_pointer_t<decltype(typed)>;
-    constexpr int V = Vec16<T>::N;
+    constexpr int V = 4;
     auto on16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     if (conv_vec<T>(a) && dim % V == 0 && k_col % V == 0 && on16(k_cache) && on16(v_cache) && on16(q_out))
       TIE_LAUNCH((conv_rope_append_kernel<T, V, 4, true>), dim3(ceil_div((q_heads + kv_heads) * (dim / V), kConvThreads), ceil_div(rows, tile)),
