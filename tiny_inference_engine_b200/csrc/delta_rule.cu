@@ -208,9 +208,9 @@ constexpr int kDeltaCols = 16;       // columns of S that a block holds
 constexpr int kDeltaPad = kDeltaCols + 1;
 constexpr int kDeltaBatch = 4;       // tokens whose read-outs are summed over the lanes together
 
-// The key channel that register r of lane `lane` (of the eight that share a column) holds: four channels in a row, then the
-// next four 32 channels on, so that a lane reads its k, q and decay entries 16 bytes at a time and the lanes of a column
-// read 128 bytes in a row (the four columns of a warp read the same 128 bytes).
+// The key channel that register r of lane `lane` (of the LANES that share a column) holds: four channels in a row, then the
+// next four 4 LANES channels on, so that a lane reads its k, q and decay entries 16 bytes at a time and the lanes of a column
+// read one piece of memory (the columns of a warp the same one).
 template <int LANES>
 __device__ __forceinline__ int delta_row(int r, int lane) { return (r >> 2) * (4 * LANES) + lane * 4 + (r & 3); }
 
@@ -227,10 +227,10 @@ struct DeltaToken {
 //                and sees its own write through a weight per key channel;  then S <- diag(g) S + k u^T
 enum DeltaMode { kDeltaRule, kDeltaPlain, kDeltaBonus };
 
-// One block per (sequence, head, 16 columns of S). A column's key channels are spread over eight lanes, R a lane. What bounds
-// the kernel is the chain from token to token: in the delta rule a product over the lane's channels, three exchanges and the
+// One block per (sequence, head, 16 columns of S). A column's key channels are spread over LANES (8 or 16) lanes, R a lane. What bounds
+// the kernel is the chain from token to token: in the delta rule a product over the lane's channels, the exchanges and the
 // update; without the correction the update alone. So everything else is kept off that chain and off the shared-memory pipe:
-// a column has few lanes (three exchanges instead of five, and one read of k, q and g serves the four columns of a warp), the
+// a column has few lanes (fewer exchanges, and the columns of a warp read the same k, q and g), the
 // read-outs of four tokens are summed over the lanes together (each exchange halves the tokens that a lane still holds), and
 // k . q of a token is formed once a chunk, for all columns. In the delta rule the read-out of the updated state is
 // (gS)^T q + (k . q) u, so it does not wait for the update.
