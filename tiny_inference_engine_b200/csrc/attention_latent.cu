@@ -14,16 +14,14 @@
 //   head_gate_mul    y[t, h, :] *= sigmoid(gate[t, h]): one gate per head.
 #include <math.h>
 
-#include "common.cuh"
+#include "rotation.cuh"
 
 namespace tie {
 
-// angle = float(pos) * inv_freq[i]; pair (i, i + rot/2).
 template <typename T>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ proj, long long stride, int q_off, int q_rank,
                                                           int kv_off, int rank, int rot, const float* __restrict__ wq,
-                                                          const float* __restrict__ wkv, float eps,
-                                                          const float* __restrict__ inv_freq,
+                                                          const float* __restrict__ wkv, float eps, Rotation turn,
                                                           const int* __restrict__ positions, const int* __restrict__ slots,
                                                           T* __restrict__ cq, T* __restrict__ k_cache) {
   pdl_sync();
@@ -51,21 +49,20 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
   inv = 1.0f / sqrtf(ss / static_cast<float>(rank) + eps);
   T* dst = k_cache + static_cast<long long>(slot) * (rank + rot);
   for (int i = threadIdx.x; i < rank; i += blockDim.x) st(dst + i, (ld(row + kv_off + i) * inv) * wkv[i]);
-  const float pos = static_cast<float>(positions[t]);
-  const int half = rot / 2;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    const float a = pos * inv_freq[i];
-    const float c = cosf(a), s = sinf(a);
-    const float u = ld(row + kv_off + rank + i), v = ld(row + kv_off + rank + half + i);
-    st(dst + rank + i, u * c - v * s);
-    st(dst + rank + half + i, v * c + u * s);
+  const int pos = positions[t];
+  for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
+    const int a = rank + turn.first(i), b = rank + turn.second(i);
+    float c, s;
+    turn.angle(pos, i, c, s);
+    const float u = ld(row + kv_off + a), v = ld(row + kv_off + b);
+    st(dst + a, u * c - v * s);
+    st(dst + b, v * c + u * s);
   }
 }
 
 template <typename T>
 __global__ void __launch_bounds__(128) latent_query_rot_kernel(const T* __restrict__ q, long long q_stride, int dim, int rot,
-                                                               const float* __restrict__ inv_freq,
-                                                               const int* __restrict__ positions, T* __restrict__ folded,
+                                                               Rotation turn, const int* __restrict__ positions, T* __restrict__ folded,
                                                                long long folded_stride, int rank, int heads,
                                                                long long items) {
   pdl_sync();
@@ -76,14 +73,14 @@ __global__ void __launch_bounds__(128) latent_query_rot_kernel(const T* __restri
   const int h = static_cast<int>(item % heads);
   const T* src = q + t * q_stride + static_cast<long long>(h) * (dim + rot) + dim;
   T* dst = folded + t * folded_stride + static_cast<long long>(h) * (rank + rot) + rank;
-  const float pos = static_cast<float>(positions[t]);
-  const int half = rot / 2;
-  for (int i = lane; i < half; i += 32) {
-    const float a = pos * inv_freq[i];
-    const float c = cosf(a), s = sinf(a);
-    const float u = ld(src + i), v = ld(src + half + i);
-    st(dst + i, u * c - v * s);
-    st(dst + half + i, v * c + u * s);
+  const int pos = positions[t];
+  for (int i = lane; i < rot / 2; i += 32) {
+    const int a = turn.first(i), b = turn.second(i);
+    float c, s;
+    turn.angle(pos, i, c, s);
+    const float u = ld(src + a), v = ld(src + b);
+    st(dst + a, u * c - v * s);
+    st(dst + b, v * c + u * s);
   }
 }
 
@@ -105,16 +102,18 @@ __global__ void head_gate_mul_kernel(T* __restrict__ y, long long y_stride, cons
 using namespace tie;
 
 TIE_API int tie_latent_prep(int dtype, const void* proj, long long stride, int q_off, int q_rank, int kv_off, int rank, int rot,
-                            const float* wq, const float* wkv, float eps, const float* inv_freq, const int* positions,
-                            const int* slots, void* cq, void* k_cache, int tokens, cudaStream_t s) {
+                            const float* wq, const float* wkv, float eps, const float* inv_freq, const double* turns, int neighbours,
+                            const int* positions, const int* slots, void* cq, void* k_cache, int tokens, cudaStream_t s) {
+  const Rotation turn{inv_freq, turns, rot, neighbours};
+  TIE_REQUIRE(rot == 0 || (inv_freq == nullptr) != (turns == nullptr), "latent_prep: a rotation takes one table of frequencies");
   TIE_REQUIRE(q_rank > 0 && rank > 0 && rot >= 0 && rot % 2 == 0, "latent_prep: bad sizes q_rank=%d rank=%d rot=%d", q_rank, rank, rot);
   if (tokens <= 0) return kOk;
   if (dtype == TIE_F32) {
     TIE_LAUNCH((latent_prep_kernel<float>), tokens, 256, 0, s, static_cast<const float*>(proj), stride, q_off, q_rank, kv_off, rank,
-               rot, wq, wkv, eps, inv_freq, positions, slots, static_cast<float*>(cq), static_cast<float*>(k_cache));
+               rot, wq, wkv, eps, turn, positions, slots, static_cast<float*>(cq), static_cast<float*>(k_cache));
   } else if (dtype == TIE_BF16) {
     TIE_LAUNCH((latent_prep_kernel<__nv_bfloat16>), tokens, 256, 0, s, static_cast<const __nv_bfloat16*>(proj), stride, q_off,
-               q_rank, kv_off, rank, rot, wq, wkv, eps, inv_freq, positions, slots, static_cast<__nv_bfloat16*>(cq),
+               q_rank, kv_off, rank, rot, wq, wkv, eps, turn, positions, slots, static_cast<__nv_bfloat16*>(cq),
                static_cast<__nv_bfloat16*>(k_cache));
   } else {
     set_error("unknown dtype code %d", dtype);
@@ -124,17 +123,19 @@ TIE_API int tie_latent_prep(int dtype, const void* proj, long long stride, int q
 }
 
 TIE_API int tie_latent_query_rot(int dtype, const void* q, long long q_stride, int dim, int rot, const float* inv_freq,
-                                 const int* positions, void* folded, long long folded_stride, int rank, int heads, int tokens,
+                                 const double* turns, int neighbours, const int* positions, void* folded, long long folded_stride, int rank, int heads, int tokens,
                                  cudaStream_t s) {
   TIE_REQUIRE(dim >= 0 && rank > 0 && rot >= 0 && rot % 2 == 0 && heads > 0, "latent_query_rot: bad sizes dim=%d rank=%d rot=%d", dim, rank, rot);
   const long long items = static_cast<long long>(tokens) * heads;
   if (items <= 0 || rot == 0) return kOk;
+  TIE_REQUIRE((inv_freq == nullptr) != (turns == nullptr), "latent_query_rot: a rotation takes one table of frequencies");
+  const Rotation turn{inv_freq, turns, rot, neighbours};
   if (dtype == TIE_F32) {
     TIE_LAUNCH((latent_query_rot_kernel<float>), ceil_div(items, 4), 128, 0, s, static_cast<const float*>(q), q_stride, dim, rot,
-               inv_freq, positions, static_cast<float*>(folded), folded_stride, rank, heads, items);
+               turn, positions, static_cast<float*>(folded), folded_stride, rank, heads, items);
   } else if (dtype == TIE_BF16) {
     TIE_LAUNCH((latent_query_rot_kernel<__nv_bfloat16>), ceil_div(items, 4), 128, 0, s, static_cast<const __nv_bfloat16*>(q),
-               q_stride, dim, rot, inv_freq, positions, static_cast<__nv_bfloat16*>(folded), folded_stride, rank, heads, items);
+               q_stride, dim, rot, turn, positions, static_cast<__nv_bfloat16*>(folded), folded_stride, rank, heads, items);
   } else {
     set_error("unknown dtype code %d", dtype);
     return kBadArgument;

@@ -30,6 +30,7 @@ struct LatentArgs {
   long long q_stride;
   int max_blocks, heads, kd, rank, page_size, window;
   float scale_log2;                // scale * log2(e)
+  const float* sink;               // [heads] or null: exp(sink[h]) is one more term of the softmax's denominator, without a value
   // sequences that bring one token, their keys cut into splits
   const int* seq_list;
   int n_list, split_keys, max_splits;
@@ -272,7 +273,11 @@ __global__ void __launch_bounds__(kLatThreads) latent_attention_mma_kernel(Laten
         dst[rank + 1] = l[half];
       }
     } else {
-      const float inv = l[half] > 0.0f ? 1.0f / l[half] : 0.0f;
+      float inv = l[half] > 0.0f ? 1.0f / l[half] : 0.0f;
+      if (a.sink != nullptr && l[half] > 0.0f) {       // sums and sink brought to the larger of the two maxima
+        const float sink = a.sink[head] * 1.4426950408889634f, top = fmaxf(m[half], sink), rescale = exp2f(m[half] - top);
+        inv = rescale / fmaf(l[half], rescale, exp2f(sink - top));
+      }
       __nv_bfloat16* dst = a.out + (static_cast<long long>(t0 + tok) * H + head) * rank;
 #pragma unroll
       for (int q = 0; q < MAXP; ++q) {
@@ -335,10 +340,10 @@ TIE_API int tie_attention_latent_mma_takes(int kd, int rank) {
 TIE_API int tie_attention_latent_prompt(const void* q, long long q_stride, const void* keys, void* out, const int* query_start,
                                         const int* context_lens, const int* block_tables, int max_blocks, int n_seqs,
                                         int max_queries, int heads, int kd, int rank, int page_size, int window, float scale,
-                                        cudaStream_t s) {
+                                        const float* sink, cudaStream_t s) {
   LatentArgs a{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(keys), static_cast<__nv_bfloat16*>(out),
                query_start, context_lens, block_tables, q_stride, max_blocks, heads, kd, rank, page_size, window,
-               scale * 1.4426950408889634f, nullptr, 0, 0, 0, nullptr};
+               scale * 1.4426950408889634f, sink, nullptr, 0, 0, 0, nullptr};
   if (const int st = check_latent(a)) return st;
   if (n_seqs <= 0 || max_queries <= 0) return kOk;
   const int hc = heads < kLatRows ? heads : kLatRows, bq = kLatRows / hc;
@@ -346,13 +351,14 @@ TIE_API int tie_attention_latent_prompt(const void* q, long long q_stride, const
   return launch_latent<false>(a, dim3(ceil_div(max_queries, bq), n_seqs, ceil_div(heads, hc)), s);
 }
 
-// Sequences of seq_list bring one token each; scratch [n_list, heads, max_splits, rank + 2] is what tie_attention_merge reads.
+// Sequences of seq_list bring one token each; scratch [n_list, heads, max_splits, rank + 2] is what tie_attention_merge
+// reads (and where a sink joins).
 TIE_API int tie_attention_latent_split(const void* q, long long q_stride, const void* keys, const int* query_start,
                                        const int* context_lens, const int* block_tables, int max_blocks, int heads, int kd,
                                        int rank, int page_size, int window, float scale, const int* seq_list, int n_list,
                                        int split_keys, int max_splits, float* scratch, cudaStream_t s) {
   LatentArgs a{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(keys), nullptr, query_start, context_lens,
-               block_tables, q_stride, max_blocks, heads, kd, rank, page_size, window, scale * 1.4426950408889634f, seq_list,
+               block_tables, q_stride, max_blocks, heads, kd, rank, page_size, window, scale * 1.4426950408889634f, nullptr, seq_list,
                n_list, split_keys, max_splits, scratch};
   if (const int st = check_latent(a)) return st;
   TIE_REQUIRE(split_keys > 0 && max_splits > 0 && max_splits <= 256 && scratch != nullptr && n_list <= 65535,

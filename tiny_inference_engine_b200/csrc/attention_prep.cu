@@ -12,7 +12,7 @@
 // to the key heads' size, so that kernels made for one head size serve it).
 #include <math.h>
 
-#include "common.cuh"
+#include "rotation.cuh"
 
 namespace tie {
 
@@ -26,8 +26,7 @@ struct PrepArgs {
   const float* wq;           // norm weights over the whole projection (null: no norm)
   const float* wk;
   float eps;
-  const float* inv_freq;     // [rot / 2] (null: no rotation)
-  int rot;
+  Rotation turn;             // of the first turn.rot dimensions of every head
   const int* positions;
   const int* slots;          // slot < 0: nothing is written to the planes
   void* k_cache;
@@ -42,7 +41,7 @@ struct PrepArgs {
 // buf[0, n) = proj + bias; then the norm over all n and the rotation, heads of `dim`.
 template <typename T>
 __device__ __forceinline__ void norm_rotate(float* buf, const T* src, const float* bias, const float* w, float eps, int n,
-                                            int dim, int rot, const float* cs, float* scratch) {
+                                            int dim, const Rotation& turn, const float* cs, float* scratch) {
   float ss = 0.0f;
   const bool wide = n % 4 == 0 && reinterpret_cast<uintptr_t>(src) % 16 == 0 && reinterpret_cast<uintptr_t>(bias) % 16 == 0;
   if (wide) {                                            // four elements a thread at a time
@@ -80,13 +79,13 @@ __device__ __forceinline__ void norm_rotate(float* buf, const T* src, const floa
   }
   __syncthreads();
   if (cs) {
-    const int half = rot / 2, heads = n / dim;
+    const int half = turn.rot / 2, heads = n / dim;
     for (int i = threadIdx.x; i < heads * half; i += blockDim.x) {
       float* h = buf + (i / half) * dim;
-      const int j = i % half;
-      const float a = h[j], b = h[j + half], c = cs[j], sn = cs[half + j];
-      h[j] = a * c - b * sn;
-      h[j + half] = b * c + a * sn;
+      const int j = i % half, j1 = turn.first(j), j2 = turn.second(j);
+      const float a = h[j1], b = h[j2], c = cs[j], sn = cs[half + j];
+      h[j1] = a * c - b * sn;
+      h[j2] = b * c + a * sn;
     }
     __syncthreads();
   }
@@ -100,19 +99,15 @@ __global__ void __launch_bounds__(256) qkv_span_prep_kernel(PrepArgs a) {
   const int t = blockIdx.x;
   const int nq = a.q_heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
   float* cs = smem;                       // [rot]
-  float* buf = smem + ((a.rot + 3) & ~3); // [max(nq, nk)], on a 16-byte boundary
+  float* buf = smem + ((a.turn.rot + 3) & ~3); // [max(nq, nk)], on a 16-byte boundary
   T* row = static_cast<T*>(a.proj) + static_cast<long long>(t) * a.stride;
-  if (a.inv_freq) {
-    const float p = static_cast<float>(a.positions[t]);
-    for (int i = threadIdx.x; i < a.rot / 2; i += blockDim.x) {
-      const float angle = p * a.inv_freq[i];
-      cs[i] = cosf(angle);
-      cs[a.rot / 2 + i] = sinf(angle);
-    }
+  if (a.turn.on()) {
+    const int p = a.positions[t];
+    for (int i = threadIdx.x; i < a.turn.rot / 2; i += blockDim.x) a.turn.angle(p, i, cs[i], cs[a.turn.rot / 2 + i]);
     __syncthreads();
   }
-  const float* table = a.inv_freq ? cs : nullptr;
-  norm_rotate<T>(buf, row + a.q_off, a.bq, a.wq, a.eps, nq, a.dim, a.rot, table, scratch);
+  const float* table = a.turn.on() ? cs : nullptr;
+  norm_rotate<T>(buf, row + a.q_off, a.bq, a.wq, a.eps, nq, a.dim, a.turn, table, scratch);
   if (nq % 4 == 0 && reinterpret_cast<uintptr_t>(row + a.q_off) % 16 == 0) {
     for (int k = 4 * threadIdx.x; k < nq; k += 4 * blockDim.x) {
       float v[4];
@@ -127,7 +122,7 @@ __global__ void __launch_bounds__(256) qkv_span_prep_kernel(PrepArgs a) {
   const int slot = a.slots[t];
   const long long page = slot >= 0 ? slot / a.page_size : 0;
   const int off = slot >= 0 ? slot % a.page_size : 0;
-  norm_rotate<T>(buf, row + a.k_off, a.bk, a.wk, a.eps, nk, a.dim, a.rot, table, scratch);
+  norm_rotate<T>(buf, row + a.k_off, a.bk, a.wk, a.eps, nk, a.dim, a.turn, table, scratch);
   if (slot >= 0) {
     T* kc = static_cast<T*>(a.k_cache);
     for (int i = threadIdx.x; i < nk; i += blockDim.x) {
@@ -158,20 +153,22 @@ using namespace tie;
 
 TIE_API int tie_qkv_span_prep(int dtype, void* proj, long long stride, int q_off, int k_off, int v_off, const float* bq,
                               const float* bk, const float* bv, const float* wq, const float* wk, float eps,
-                              const float* inv_freq, int rot, const int* positions, const int* slots, void* k_cache,
+                              const float* inv_freq, const double* turns, int rot, int neighbours, const int* positions, const int* slots, void* k_cache,
                               void* v_cache, int tokens, int q_heads, int kv_heads, int dim, int vdim, int v_plane,
                               int page_size, int mix_mode, float* v_first, const float* lambda, cudaStream_t s) {
   TIE_REQUIRE(v_plane >= vdim, "qkv_span_prep: rows of the value plane (%d) are narrower than a value head (%d)", v_plane, vdim);
   TIE_REQUIRE(tokens >= 0 && q_heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && page_size > 0,
               "qkv_span_prep: bad sizes tokens=%d heads=%d/%d dim=%d vdim=%d page=%d", tokens, q_heads, kv_heads, dim, vdim,
               page_size);
-  TIE_REQUIRE(inv_freq == nullptr || (rot > 0 && rot % 2 == 0 && rot <= dim), "qkv_span_prep: %d rotated dimensions of a head of %d",
+  TIE_REQUIRE(inv_freq == nullptr || turns == nullptr, "qkv_span_prep: a rotation takes one table of frequencies");
+  const bool turned = inv_freq != nullptr || turns != nullptr;
+  TIE_REQUIRE(!turned || (rot > 0 && rot % 2 == 0 && rot <= dim), "qkv_span_prep: %d rotated dimensions of a head of %d",
               rot, dim);
   TIE_REQUIRE(mix_mode == 0 || (v_first != nullptr && (mix_mode == 1 || (mix_mode == 2 && lambda != nullptr))),
               "qkv_span_prep: value blending (mode %d) needs the first values and, to blend, its weight", mix_mode);
   if (tokens == 0) return kOk;
-  if (inv_freq == nullptr) rot = 0;
-  const PrepArgs a{proj, stride, q_off, k_off, v_off, bq, bk, bv, wq, wk, eps, inv_freq, rot, positions, slots, k_cache,
+  if (!turned) rot = 0;
+  const PrepArgs a{proj, stride, q_off, k_off, v_off, bq, bk, bv, wq, wk, eps, Rotation{inv_freq, turns, rot, neighbours}, positions, slots, k_cache,
                    v_cache, q_heads, kv_heads, dim, vdim, page_size, v_plane, mix_mode, v_first, lambda};
   const int widest = q_heads * dim > kv_heads * dim ? q_heads * dim : kv_heads * dim;
   const size_t smem = static_cast<size_t>(((rot + 3) & ~3) + widest) * sizeof(float);

@@ -596,10 +596,11 @@ TIE_API int tie_attention_split(int dtype, const void* q, long long q_stride, co
 }
 
 // Combines the (acc, max, sum) that a split kernel (this file's or the tensor-core one) left in
-// scratch [n_list, q_heads, max_splits, head_dim + 2] into out rows, in split order.
+// scratch [n_list, q_heads, max_splits, head_dim + 2] into out rows, in split order. `sink` (float [q_heads] or null):
+// exp(sink[h]) is one more term of head h's denominator.
 TIE_API int tie_attention_merge(int dtype, void* out, const int* query_start, const int* context_lens, int q_heads,
                                 int head_dim, int window, const int* seq_list, int n_list, int split_keys, int max_splits,
-                                const float* scratch, cudaStream_t s) {
+                                const float* scratch, const float* sink, cudaStream_t s) {
   TIE_REQUIRE(q_heads > 0 && head_dim > 0 && split_keys > 0 && max_splits > 0 && max_splits <= kMergeMaxSplits,
               "attention merge: bad geometry (at most %d splits)", kMergeMaxSplits);
   if (n_list == 0) return kOk;
@@ -610,6 +611,7 @@ TIE_API int tie_attention_merge(int dtype, void* out, const int* query_start, co
   a.q_heads = q_heads;
   a.head_dim = head_dim;
   a.window = window;
+  a.sink = sink;
   const long long items = static_cast<long long>(n_list) * q_heads;
   if (dtype == TIE_F32) {
     TIE_LAUNCH((attention_merge_kernel<float>), static_cast<int>(items), kMergeThreads, 0, s, a, seq_list, n_list, split_keys, max_splits, scratch);
@@ -623,14 +625,16 @@ TIE_API int tie_attention_merge(int dtype, void* out, const int* query_start, co
 }
 
 // The same two for keys and values of different head sizes: queries and keys have head_dim, values and the
-// output v_dim (planes [pages, kv_heads, page_size, head_dim] and [pages, kv_heads, page_size, v_dim]).
+// output v_dim (planes [pages, kv_heads, page_size, head_dim] and [pages, kv_heads, page_size, v_dim]), with an optional sink
+// per head in the softmax.
 TIE_API int tie_attention_rows_dv(int dtype, const void* q, long long q_stride, const void* k_cache, const void* v_cache,
                                   void* out, const int* seq_of_row, const int* query_start, const int* context_lens,
                                   const int* block_tables, int max_blocks, int rows, int seqs, int q_heads, int kv_heads,
-                                  int head_dim, int v_dim, int page_size, int window, float scale, int v_ld,
+                                  int head_dim, int v_dim, int page_size, int window, float scale, int v_ld, const float* sink,
                                   cudaStream_t s) {
-  const AttnArgs a{q, k_cache, v_cache, out, seq_of_row, query_start, context_lens, block_tables, q_stride, max_blocks,
+  AttnArgs a{q, k_cache, v_cache, out, seq_of_row, query_start, context_lens, block_tables, q_stride, max_blocks,
                    rows, seqs, q_heads, kv_heads, head_dim, page_size, window, scale, v_dim, v_ld};
+  a.sink = sink;
   TIE_REQUIRE(v_ld == 0 || v_ld >= v_dim, "attention: value rows %d apart are shorter than a value head of %d", v_ld, v_dim);
   if (const int st = check_attn(a, true)) return st;
   if (dtype == TIE_F32) return launch_attention<float>(a, nullptr, nullptr, 0, 0, 0, nullptr, 1, s);
@@ -643,9 +647,10 @@ TIE_API int tie_attention_split_dv(int dtype, const void* q, long long q_stride,
                                    void* out, const int* query_start, const int* context_lens, const int* block_tables,
                                    int max_blocks, int seqs, int q_heads, int kv_heads, int head_dim, int v_dim,
                                    int page_size, int window, float scale, const int* seq_list, int n_list, int split_keys,
-                                   int max_splits, float* scratch, int v_ld, cudaStream_t s) {
-  const AttnArgs a{q, k_cache, v_cache, out, nullptr, query_start, context_lens, block_tables, q_stride, max_blocks,
+                                   int max_splits, float* scratch, int v_ld, const float* sink, cudaStream_t s) {
+  AttnArgs a{q, k_cache, v_cache, out, nullptr, query_start, context_lens, block_tables, q_stride, max_blocks,
                    0, seqs, q_heads, kv_heads, head_dim, page_size, window, scale, v_dim, v_ld};
+  a.sink = sink;
   TIE_REQUIRE(v_ld == 0 || v_ld >= v_dim, "attention: value rows %d apart are shorter than a value head of %d", v_ld, v_dim);
   if (const int st = check_attn(a, true)) return st;
   TIE_REQUIRE(split_keys > 0 && max_splits > 0 && max_splits <= kMergeMaxSplits && scratch != nullptr,

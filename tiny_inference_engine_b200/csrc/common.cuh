@@ -110,6 +110,14 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   return scratch[32];
 }
 
+// The epilogues of a product (`silu` in the launchers): 1 and 2 a gated unit, act(gate) * up with the SiLU or the ReLU, over weight
+// rows in blocks of 16 gate rows and their 16 up rows; 3 the squared ReLU of every output.
+constexpr int kEpilogueSquaredRelu = 3;
+__device__ __forceinline__ float squared_relu(float v) {
+  const float r = fmaxf(v, 0.0f);
+  return r * r;
+}
+
 // The activation of a gated product's epilogue: 1 the SiLU, 2 the ReLU.
 __device__ __forceinline__ float gate_act(float g, int act) { return act == 2 ? fmaxf(g, 0.0f) : g / (1.0f + expf(-g)); }
 

@@ -9,6 +9,7 @@
 #include "common.cuh"
 #include "head_prep.cuh"
 #include "launchers.h"
+#include "rotation.cuh"
 
 namespace tie {
 
@@ -285,24 +286,24 @@ __global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, i
 }
 
 // ---------------------------------------------------------------------------------------------
-// Rotate-half RoPE in place over the first `rot` dims of every head:
-//   angle = float(pos) * inv_freq[i];  (v[i], v[i + rot/2]) <- (v[i] c - v[i+rot/2] s, v[i+rot/2] c + v[i] s)
+// RoPE in place over the first `rot` dims of every head, (u, v) <- (u c - v s, v c + u s) for the pairs and angles of `turn`.
 template <typename T>
 __global__ void rope_kernel(T* __restrict__ x, long long row_stride, const int* __restrict__ positions,
-                            const float* __restrict__ inv_freq, int heads, int head_dim, int rot, long long total) {
+                            Rotation turn, int heads, int head_dim, long long total) {
   pdl_sync();
   const long long idx = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (idx >= total) return;
-  const int half = rot / 2;
+  const int half = turn.rot / 2;
   const int i = static_cast<int>(idx % half);
   const int h = static_cast<int>((idx / half) % heads);
   const long long t = idx / (static_cast<long long>(half) * heads);
   T* v = x + t * row_stride + static_cast<long long>(h) * head_dim;
-  const float angle = static_cast<float>(positions[t]) * inv_freq[i];
-  const float c = cosf(angle), s = sinf(angle);
-  const float x1 = ld(v + i), x2 = ld(v + i + half);
-  st(v + i, x1 * c - x2 * s);
-  st(v + i + half, x2 * c + x1 * s);
+  float c, s;
+  turn.angle(positions[t], i, c, s);
+  T *p1 = v + turn.first(i), *p2 = v + turn.second(i);
+  const float x1 = ld(p1), x2 = ld(p2);
+  st(p1, x1 * c - x2 * s);
+  st(p2, x2 * c + x1 * s);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -651,12 +652,11 @@ int launch_silu_mul(const void* gu, void* out, int tokens, int inter, cudaStream
 }
 
 template <typename T>
-int launch_rope(void* x, long long stride, const int* pos, const float* inv_freq, int tokens, int heads, int head_dim,
-                int rot, cudaStream_t s) {
-  const long long total = static_cast<long long>(tokens) * heads * (rot / 2);
+int launch_rope(void* x, long long stride, const int* pos, const Rotation& turn, int tokens, int heads, int head_dim,
+                cudaStream_t s) {
+  const long long total = static_cast<long long>(tokens) * heads * (turn.rot / 2);
   if (total == 0) return kOk;
-  TIE_LAUNCH((rope_kernel<T>), ceil_div(total, 256), 256, 0, s, static_cast<T*>(x), stride, pos, inv_freq, heads, head_dim, rot,
-                                                      total);
+  TIE_LAUNCH((rope_kernel<T>), ceil_div(total, 256), 256, 0, s, static_cast<T*>(x), stride, pos, turn, heads, head_dim, total);
   TIE_RETURN_LAUNCH("rope");
 }
 
@@ -794,12 +794,14 @@ TIE_API int tie_silu_mul(int dtype, const void* gu, void* out, int tokens, int i
                launch_silu_mul<__nv_bfloat16>(gu, out, tokens, inter, s));
 }
 
-TIE_API int tie_rope(int dtype, void* x, long long stride, const int* pos, const float* inv_freq, int tokens,
+TIE_API int tie_rope(int dtype, void* x, long long stride, const int* pos, const float* inv_freq, const double* turns, int neighbours, int tokens,
                      int heads, int head_dim, int rot, cudaStream_t s) {
   TIE_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= head_dim, "rope: rotary dim %d must be even and at most head_dim %d",
               rot, head_dim);
-  TIE_DISPATCH(dtype, launch_rope<float>(x, stride, pos, inv_freq, tokens, heads, head_dim, rot, s),
-               launch_rope<__nv_bfloat16>(x, stride, pos, inv_freq, tokens, heads, head_dim, rot, s));
+  TIE_REQUIRE((inv_freq == nullptr) != (turns == nullptr), "rope: a rotation takes one table of frequencies");
+  const Rotation turn{inv_freq, turns, rot, neighbours};
+  TIE_DISPATCH(dtype, launch_rope<float>(x, stride, pos, turn, tokens, heads, head_dim, s),
+               launch_rope<__nv_bfloat16>(x, stride, pos, turn, tokens, heads, head_dim, s));
 }
 
 TIE_API int tie_kv_append(int dtype, const void* k, const void* v, long long k_stride, long long v_stride,

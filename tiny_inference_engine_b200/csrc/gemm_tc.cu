@@ -228,7 +228,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t tmem_acc = tmem_base + buf * BN;
       const int i = i0 + warp * 32 + lane;
-      if (silu) {
+      if (silu != 0 && silu != kEpilogueSquaredRelu) {
         // The weight rows come in blocks of 16 gate rows followed by their 16 up rows; the output is
         // act(gate) * up (act 1: the SiLU, 2: the ReLU), half as wide as the product: out[token, 16 * block + r].
         if (transposed) {
@@ -292,6 +292,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           uint32_t r[16];
           tmem_ld16(tmem_acc + (static_cast<uint32_t>(warp * 32) << 16) + c0, r);
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+          if (silu == kEpilogueSquaredRelu && part == nullptr) {      // (with split k the reduce kernel applies it)
+#pragma unroll
+            for (int e = 0; e < 16; ++e) r[e] = __float_as_uint(squared_relu(__uint_as_float(r[e])));
+          }
           if (i < rows_x) {
             if (transposed) {
 #pragma unroll
@@ -358,13 +362,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
 // out[m, n] = sum over splits of partial[z][m, n], in split order, converted to OutT.
 template <typename OutT>
 __global__ void splitk_reduce_kernel(const float* __restrict__ partial, long long part_stride, int splits,
-                                     OutT* __restrict__ out, long long ldo, int N, long long total) {
+                                     OutT* __restrict__ out, long long ldo, int N, long long total, int epilogue) {
   pdl_sync();
   const long long idx = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (idx >= total) return;
   float acc = partial[idx];
   for (int z = 1; z < splits; ++z) acc += partial[static_cast<long long>(z) * part_stride + idx];
-  st(out + (idx / N) * ldo + idx % N, acc);
+  st(out + (idx / N) * ldo + idx % N, epilogue == kEpilogueSquaredRelu ? squared_relu(acc) : acc);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -409,7 +413,8 @@ using namespace tie;
 // with tie_gemm_tc_scratch_floats floats: the float partial sums [splits, M, N]; with reduce == 0
 // they are left there for a consumer that adds them itself (tie_gemm_tc_real_splits says how
 // many there are). silu != 0: w holds blocks of 16 gate rows followed by their 16 up rows and
-// out[M, N / 2] = act(gate) * up, act the SiLU (1) or the ReLU (2). deep != 0: the deepest shared-memory ring (one CTA per SM), else
+// out[M, N / 2] = act(gate) * up, act the SiLU (1) or the ReLU (2); silu == 3: out[M, N] = max(product, 0)^2, with split k
+// applied by the reduction (reduce != 0). deep != 0: the deepest shared-memory ring (one CTA per SM), else
 // a ring of about 100 KB (two CTAs per SM). Returns kBadArgument
 // with a message for sizes it does not take (K or a row stride not a multiple of 8, unaligned
 // pointers): the caller then uses the CUDA-core kernel.
@@ -436,7 +441,9 @@ TIE_API int tie_gemm_tc(int out_dtype, const void* a, const void* w, void* out, 
   TIE_REQUIRE(bn == 16 || bn == 32 || bn == 64 || bn == 128 || bn == 256, "gemm_tc: tile width %d", bn);
   TIE_REQUIRE(splits >= 1 && (splits == 1 || scratch != nullptr), "gemm_tc: splits=%d needs scratch memory", splits);
   TIE_REQUIRE(out_dtype == TIE_BF16 || out_dtype == TIE_F32, "gemm_tc: output dtype code %d", out_dtype);
-  TIE_REQUIRE(!silu || (splits == 1 && N % 32 == 0 && (transposed || bn >= 32)),
+  TIE_REQUIRE(silu >= 0 && silu <= kEpilogueSquaredRelu && (silu != kEpilogueSquaredRelu || splits == 1 || reduce),
+              "gemm_tc: epilogue %d (the squared ReLU of a split product needs the reduction here)", silu);
+  TIE_REQUIRE(silu == 0 || silu == kEpilogueSquaredRelu || (splits == 1 && N % 32 == 0 && (transposed || bn >= 32)),
               "gemm_tc: the SiLU epilogue needs unsplit k and weight rows in blocks of 16 gate + 16 up (N=%d)", N);
   TIE_REQUIRE(status_word() != nullptr, "gemm_tc: cannot allocate the status word");
   // row operand X (128 per tile) and column operand Y (bn per tile)
@@ -478,10 +485,10 @@ TIE_API int tie_gemm_tc(int out_dtype, const void* a, const void* w, void* out, 
     const long long total = part_stride;
     if (out_dtype == TIE_BF16) {
       TIE_LAUNCH((splitk_reduce_kernel<__nv_bfloat16>), ceil_div(total, 256), 256, 0, s, 
-          partial, part_stride, real_splits, static_cast<__nv_bfloat16*>(out), ldo, N, total);
+          partial, part_stride, real_splits, static_cast<__nv_bfloat16*>(out), ldo, N, total, silu);
     } else {
       TIE_LAUNCH((splitk_reduce_kernel<float>), ceil_div(total, 256), 256, 0, s, partial, part_stride, real_splits,
-                                                                      static_cast<float*>(out), ldo, N, total);
+                                                                      static_cast<float*>(out), ldo, N, total, silu);
     }
   }
   TIE_RETURN_LAUNCH("gemm_tc");

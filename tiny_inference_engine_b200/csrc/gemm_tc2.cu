@@ -215,7 +215,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t tmem_acc = tmem_base + buf * 256;
       const int i = i0 + warp * 32 + lane;
-      if (silu) {
+      if (silu != 0 && silu != kEpilogueSquaredRelu) {
 #pragma unroll 1
         for (int c0 = 0; c0 < BN; c0 += 32) {
           if (j0 + c0 >= N) break;
@@ -253,6 +253,10 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
           uint32_t r[16];
           tmem_ld16(tmem_acc + (static_cast<uint32_t>(warp * 32) << 16) + c0, r);
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+          if (silu == kEpilogueSquaredRelu) {
+#pragma unroll
+            for (int e = 0; e < 16; ++e) r[e] = __float_as_uint(squared_relu(__uint_as_float(r[e])));
+          }
           if (i < M) {
             const long long at = static_cast<long long>(i) * ldo + j0 + c0;
             const int n = min(16, N - (j0 + c0));
@@ -375,7 +379,8 @@ static int launch_tc2(const CUtensorMap& ma, const CUtensorMap& mw, void* out, i
 
 using namespace tie;
 
-// out[M, N] (or, with silu 1 or 2, out[M, N / 2] = act(gate) * up, act the SiLU or the ReLU, for w in blocks of 16 gate + 16 up rows)
+// out[M, N] (or, with silu 1 or 2, out[M, N / 2] = act(gate) * up, act the SiLU or the ReLU, for w in blocks of 16 gate + 16 up
+// rows; with 3, out[M, N] = max(product, 0)^2)
 // = a[M, K] . w[N, K]^T on pairs of SMs. a, w bfloat16 with K and row strides multiples of 8. w_rows > 0: w is
 // stored in k-blocks, [ceil(K / 64)][w_rows][64], and the product uses its rows w_row0 .. w_row0 + N - 1 (gemm_tc.cu).
 // How many pairs of SMs hold the kernel at once: what the host counts waves of tiles with.
@@ -392,7 +397,8 @@ TIE_API int tie_gemm_tc2(int out_dtype, const void* a, const void* w, void* out,
   TIE_REQUIRE(reinterpret_cast<uintptr_t>(a) % 16 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0,
               "gemm_tc2: operands must be 16-byte aligned");
   TIE_REQUIRE(out_dtype == TIE_BF16 || out_dtype == TIE_F32, "gemm_tc2: output dtype code %d", out_dtype);
-  TIE_REQUIRE(!silu || N % 32 == 0, "gemm_tc2: the SiLU epilogue needs weight rows in blocks of 16 gate + 16 up (N=%d)", N);
+  TIE_REQUIRE(silu >= 0 && silu <= kEpilogueSquaredRelu, "gemm_tc2: epilogue %d", silu);
+  TIE_REQUIRE(silu == 0 || silu == kEpilogueSquaredRelu || N % 32 == 0, "gemm_tc2: the SiLU epilogue needs weight rows in blocks of 16 gate + 16 up (N=%d)", N);
   TIE_REQUIRE(status_word() != nullptr, "gemm_tc2: cannot allocate the status word");
   CUtensorMap ma, mw;
   const bool w_ok = w_rows > 0 ? make_map_bf16(&mw, w, static_cast<long long>(ceil_div(K, k2BK)) * w_rows, k2BK, k2BK, k2BK, bn / 2)

@@ -13,7 +13,7 @@ TIE_API int tie_add_rmsnorm(int dtype, float* x, const void* delta, const float*
 TIE_API int tie_rmsnorm_rows(int dtype, const void* x, long long x_stride, const float* w, float eps, void* out,
                              long long out_stride, int size, long long n, cudaStream_t s);
 TIE_API int tie_silu_mul(int dtype, const void* gu, void* out, int tokens, int inter, cudaStream_t s);
-TIE_API int tie_rope(int dtype, void* x, long long stride, const int* pos, const float* inv_freq, int tokens,
+TIE_API int tie_rope(int dtype, void* x, long long stride, const int* pos, const float* inv_freq, const double* turns, int neighbours, int tokens,
                      int heads, int head_dim, int rot, cudaStream_t s);
 TIE_API int tie_kv_append(int dtype, const void* k, const void* v, long long k_stride, long long v_stride,
                           const int* slots, void* k_cache, void* v_cache, int tokens, int kv_heads, int head_dim,
@@ -43,7 +43,7 @@ TIE_API int tie_attention_split(int dtype, const void* q, long long q_stride, co
                                 int max_splits, float* scratch, cudaStream_t s);
 TIE_API int tie_attention_merge(int dtype, void* out, const int* query_start, const int* context_lens, int q_heads,
                                 int head_dim, int window, const int* seq_list, int n_list, int split_keys, int max_splits,
-                                const float* scratch, cudaStream_t s);
+                                const float* scratch, const float* sink, cudaStream_t s);
 TIE_API int tie_attention_prompt_tc(const void* q, long long q_stride, const void* k_cache, const void* v_cache, void* out,
                                     const int* query_start, const int* context_lens, const int* block_tables,
                                     int max_blocks, int n_seqs, int max_queries, int q_heads, int kv_heads, int head_dim,

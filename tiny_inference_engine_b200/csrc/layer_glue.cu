@@ -4,6 +4,7 @@
 //                       the residual add of a sublayer whose output passes a norm of its own first, fused with
 //                       the norm ahead of the next sublayer. All of it in float: y, both sums, the residual.
 //   glu_clamped         out = g' * sigmoid(slope * g') * (u' + up_shift),  g' = min(g, limit), u' = clamp(u, +-limit)
+//   two_branch_unit, squared_relu  activations of a feed-forward without a gate
 //   sigmoid_gate_mul    y *= sigmoid(gate)  (a gate on the heads' outputs)
 //   scale_rows          x *= c  (float rows: the logits of a model that scales them)
 #include <math.h>
@@ -152,23 +153,27 @@ __global__ void glu_clamped_kernel(const T* __restrict__ gu, T* __restrict__ out
   st(out + i, (g / (1.0f + expf(-slope * g))) * (u + up_shift));
 }
 
-// One hidden layer's activation in two branches that meet at zero with the slope 1/2:
-//   z > 0: c_pos z^2 + z / 2;   z <= 0: c_neg (exp(z) - 1 - z) + z / 2.
-__device__ __forceinline__ float two_branch(float v, float c_pos, float c_neg) {
-  return v > 0.0f ? fmaf(c_pos * v, v, 0.5f * v) : fmaf(c_neg, expm1f(v) - v, 0.5f * v);
-}
+// Activations of a feed-forward with one hidden layer and no gate.
+// Two branches that meet at zero with the slope 1/2: z > 0: c_pos z^2 + z / 2;   z <= 0: c_neg (exp(z) - 1 - z) + z / 2.
+struct TwoBranch {
+  float c_pos, c_neg;
+  __device__ __forceinline__ float operator()(float v) const { return v > 0.0f ? fmaf(c_pos * v, v, 0.5f * v) : fmaf(c_neg, expm1f(v) - v, 0.5f * v); }
+};
+struct SquaredRelu {      // max(z, 0)^2
+  __device__ __forceinline__ float operator()(float v) const { return squared_relu(v); }
+};
 
-template <typename T>
-__global__ void two_branch_unit_kernel(const T* __restrict__ z, T* __restrict__ out, long long total, float c_pos, float c_neg) {
+template <typename T, typename F>
+__global__ void unit_kernel(const T* __restrict__ z, T* __restrict__ out, long long total, F act) {
   pdl_sync();
   const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= total) return;
-  st(out + i, two_branch(ld(z + i), c_pos, c_neg));
+  st(out + i, act(ld(z + i)));
 }
 
 // 16 bytes a thread.
-template <typename T>
-__global__ void two_branch_unit_vec_kernel(const T* __restrict__ z, T* __restrict__ out, long long pieces, float c_pos, float c_neg) {
+template <typename T, typename F>
+__global__ void unit_vec_kernel(const T* __restrict__ z, T* __restrict__ out, long long pieces, F act) {
   pdl_sync();
   constexpr int V = Vec16<T>::N;
   const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
@@ -176,8 +181,34 @@ __global__ void two_branch_unit_vec_kernel(const T* __restrict__ z, T* __restric
   Vec16<T> v;
   v.load(z + i * V);
 #pragma unroll
-  for (int e = 0; e < V; ++e) v.v[e] = two_branch(v.v[e], c_pos, c_neg);
+  for (int e = 0; e < V; ++e) v.v[e] = act(v.v[e]);
   v.store(out + i * V);
+}
+
+template <typename T, typename F>
+void launch_unit(const void* z, void* out, long long total, F act, cudaStream_t s) {
+  constexpr int V = Vec16<T>::N;
+  const T* in = static_cast<const T*>(z);
+  T* o = static_cast<T*>(out);
+  if (reinterpret_cast<uintptr_t>(z) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0 && total % V == 0)
+    TIE_LAUNCH((unit_vec_kernel<T, F>), ceil_div(total / V, 256), 256, 0, s, in, o, total / V, act);
+  else
+    TIE_LAUNCH((unit_kernel<T, F>), ceil_div(total, 256), 256, 0, s, in, o, total, act);
+}
+
+template <typename F>
+int launch_unit_of(int dtype, const void* z, void* out, long long total, F act, const char* name, cudaStream_t s) {
+  TIE_REQUIRE(total >= 0, "%s: bad size", name);
+  if (total == 0) return kOk;
+  if (dtype == TIE_F32) {
+    launch_unit<float>(z, out, total, act, s);
+  } else if (dtype == TIE_BF16) {
+    launch_unit<__nv_bfloat16>(z, out, total, act, s);
+  } else {
+    set_error("unknown dtype code %d", dtype);
+    return kBadArgument;
+  }
+  TIE_RETURN_LAUNCH(name);
 }
 
 template <typename T>
@@ -323,28 +354,11 @@ TIE_API int tie_glu_clamped(int dtype, const void* gu, void* out, int tokens, in
 }
 
 TIE_API int tie_two_branch_unit(int dtype, const void* z, void* out, long long total, float c_pos, float c_neg, cudaStream_t s) {
-  TIE_REQUIRE(total >= 0, "two_branch_unit: bad size");
-  if (total == 0) return kOk;
-  const bool aligned = reinterpret_cast<uintptr_t>(z) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0;
-  if (dtype == TIE_F32) {
-    if (aligned && total % 4 == 0)
-      TIE_LAUNCH((two_branch_unit_vec_kernel<float>), ceil_div(total / 4, 256), 256, 0, s, static_cast<const float*>(z), static_cast<float*>(out),
-                 total / 4, c_pos, c_neg);
-    else
-      TIE_LAUNCH((two_branch_unit_kernel<float>), ceil_div(total, 256), 256, 0, s, static_cast<const float*>(z), static_cast<float*>(out), total,
-                 c_pos, c_neg);
-  } else if (dtype == TIE_BF16) {
-    if (aligned && total % 8 == 0)
-      TIE_LAUNCH((two_branch_unit_vec_kernel<__nv_bfloat16>), ceil_div(total / 8, 256), 256, 0, s, static_cast<const __nv_bfloat16*>(z),
-                 static_cast<__nv_bfloat16*>(out), total / 8, c_pos, c_neg);
-    else
-      TIE_LAUNCH((two_branch_unit_kernel<__nv_bfloat16>), ceil_div(total, 256), 256, 0, s, static_cast<const __nv_bfloat16*>(z),
-                 static_cast<__nv_bfloat16*>(out), total, c_pos, c_neg);
-  } else {
-    set_error("unknown dtype code %d", dtype);
-    return kBadArgument;
-  }
-  TIE_RETURN_LAUNCH("two_branch_unit");
+  return launch_unit_of(dtype, z, out, total, TwoBranch{c_pos, c_neg}, "two_branch_unit", s);
+}
+
+TIE_API int tie_squared_relu(int dtype, const void* z, void* out, long long total, cudaStream_t s) {
+  return launch_unit_of(dtype, z, out, total, SquaredRelu{}, "squared_relu", s);
 }
 
 TIE_API int tie_sigmoid_gate_mul(int dtype, void* y, long long y_stride, const void* gate, long long gate_stride, int tokens,

@@ -1,10 +1,12 @@
-// A norm with mean and variance, and sums into the residual stream outside a norm.
+// Norms that add a sum of sublayer outputs to the residual stream on their way (with mean and variance, or by the root mean
+// square), and sums into the stream outside a norm.
 //
 //   add_layer_norm   x += the terms (float, in place, added in order; up to four, each a tensor in the compute type or the
 //                    partial sums of a split product, times a factor), then
 //                    out = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b in the compute type. With `rows`, out[i]
 //                    comes from row rows[i] and x is left as it is. One block a row: the row stays in registers between
 //                    the sum of the terms, the mean and the squared deviations.
+//   add_terms_rmsnorm  the same without a mean and a bias: out = x / sqrt(mean(x^2) + eps) * w.
 //   stream_add       x += the terms, then + other (float rows), then + vec (one float row for every row); any may be absent.
 #include <math.h>
 
@@ -12,7 +14,8 @@
 
 namespace tie {
 
-template <typename T, int NV>
+// CENTER: with mean and bias; otherwise the root mean square alone.
+template <typename T, int NV, bool CENTER>
 __global__ void __launch_bounds__(1024) add_layer_norm_vec4_kernel(float* __restrict__ x, Terms terms, const int* __restrict__ rows,
                                                                    const float* __restrict__ w, const float* __restrict__ bias, float eps,
                                                                    T* __restrict__ out, int D) {
@@ -28,17 +31,17 @@ __global__ void __launch_bounds__(1024) add_layer_norm_vec4_kernel(float* __rest
       load4(x + r * D + d, v[i]);
       for (int k = 0; k < terms.n; ++k) term_add4<T>(terms.t[k], r * D + d, v[i]);
       if (rows == nullptr && terms.n > 0) store4(x + r * D + d, v[i]);
-      sum += (v[i][0] + v[i][1]) + (v[i][2] + v[i][3]);
+      if constexpr (CENTER) sum += (v[i][0] + v[i][1]) + (v[i][2] + v[i][3]);
     }
   }
-  const float mean = block_sum(sum, scratch) / static_cast<float>(D);
+  const float mean = CENTER ? block_sum(sum, scratch) / static_cast<float>(D) : 0.0f;
   float ss = 0.0f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     if ((threadIdx.x + i * blockDim.x) * 4 < D) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        v[i][e] -= mean;
+        if constexpr (CENTER) v[i][e] -= mean;
         ss = fmaf(v[i][e], v[i][e], ss);
       }
     }
@@ -50,16 +53,16 @@ __global__ void __launch_bounds__(1024) add_layer_norm_vec4_kernel(float* __rest
     if (d < D) {
       float ww[4], bb[4], o[4];
       load4(w + d, ww);
-      load4(bias + d, bb);
+      if constexpr (CENTER) load4(bias + d, bb);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) o[e] = fmaf(v[i][e] * inv, ww[e], bb[e]);
+      for (int e = 0; e < 4; ++e) o[e] = CENTER ? fmaf(v[i][e] * inv, ww[e], bb[e]) : (v[i][e] * inv) * ww[e];
       store4(out + static_cast<long long>(blockIdx.x) * D + d, o);
     }
   }
 }
 
 // Any width: the row waits in shared memory.
-template <typename T>
+template <typename T, bool CENTER>
 __global__ void __launch_bounds__(256) add_layer_norm_kernel(float* __restrict__ x, Terms terms, const int* __restrict__ rows,
                                                              const float* __restrict__ w, const float* __restrict__ bias, float eps,
                                                              T* __restrict__ out, int D) {
@@ -75,7 +78,7 @@ __global__ void __launch_bounds__(256) add_layer_norm_kernel(float* __restrict__
     row[d] = v;
     sum += v;
   }
-  const float mean = block_sum(sum, scratch) / static_cast<float>(D);
+  const float mean = CENTER ? block_sum(sum, scratch) / static_cast<float>(D) : 0.0f;
   float ss = 0.0f;
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
     const float v = row[d] - mean;
@@ -83,7 +86,7 @@ __global__ void __launch_bounds__(256) add_layer_norm_kernel(float* __restrict__
   }
   const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(D) + eps);
   for (int d = threadIdx.x; d < D; d += blockDim.x)
-    st(out + static_cast<long long>(blockIdx.x) * D + d, fmaf((row[d] - mean) * inv, w[d], bias[d]));
+    st(out + static_cast<long long>(blockIdx.x) * D + d, CENTER ? fmaf((row[d] - mean) * inv, w[d], bias[d]) : (row[d] * inv) * w[d]);
 }
 
 template <typename T>
@@ -134,7 +137,7 @@ static Terms pack_terms(TIE_TERMS) {
   return terms;
 }
 
-template <typename T>
+template <typename T, bool CENTER>
 static int launch_add_layer_norm(float* x, const Terms& terms, const int* rows, const float* w, const float* bias, float eps, void* out,
                                  int n, int D, cudaStream_t s) {
   T* o = static_cast<T*>(out);
@@ -145,20 +148,20 @@ static int launch_add_layer_norm(float* x, const Terms& terms, const int* rows, 
     while (threads < 1024 && pieces > 4 * threads) threads *= 2;
     while (threads > 32 && threads / 2 >= pieces) threads /= 2;
     const int nv = (pieces + threads - 1) / threads;
-    if (nv <= 1) TIE_LAUNCH((add_layer_norm_vec4_kernel<T, 1>), n, threads, 0, s, x, terms, rows, w, bias, eps, o, D);
-    else if (nv <= 2) TIE_LAUNCH((add_layer_norm_vec4_kernel<T, 2>), n, threads, 0, s, x, terms, rows, w, bias, eps, o, D);
-    else TIE_LAUNCH((add_layer_norm_vec4_kernel<T, 4>), n, threads, 0, s, x, terms, rows, w, bias, eps, o, D);
+    if (nv <= 1) TIE_LAUNCH((add_layer_norm_vec4_kernel<T, 1, CENTER>), n, threads, 0, s, x, terms, rows, w, bias, eps, o, D);
+    else if (nv <= 2) TIE_LAUNCH((add_layer_norm_vec4_kernel<T, 2, CENTER>), n, threads, 0, s, x, terms, rows, w, bias, eps, o, D);
+    else TIE_LAUNCH((add_layer_norm_vec4_kernel<T, 4, CENTER>), n, threads, 0, s, x, terms, rows, w, bias, eps, o, D);
     TIE_RETURN_LAUNCH("add_layer_norm");
   }
   const size_t smem = static_cast<size_t>(D) * sizeof(float);
   TIE_REQUIRE(smem <= 200 * 1024, "add_layer_norm: a row of %d exceeds the kernel's shared memory", D);
   if (smem > 48 * 1024) {
-    if (cudaFuncSetAttribute(add_layer_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess) {
+    if (cudaFuncSetAttribute(add_layer_norm_kernel<T, CENTER>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess) {
       set_error("add_layer_norm: cannot reserve %zu bytes of shared memory", smem);
       return kCudaError;
     }
   }
-  TIE_LAUNCH((add_layer_norm_kernel<T>), n, 256, smem, s, x, terms, rows, w, bias, eps, o, D);
+  TIE_LAUNCH((add_layer_norm_kernel<T, CENTER>), n, 256, smem, s, x, terms, rows, w, bias, eps, o, D);
   TIE_RETURN_LAUNCH("add_layer_norm");
 }
 
@@ -167,8 +170,19 @@ TIE_API int tie_add_layer_norm(int dtype, float* x, TIE_TERMS, const int* rows, 
   TIE_REQUIRE(n >= 0 && D > 0, "add_layer_norm: bad sizes n=%d D=%d", n, D);
   if (n == 0) return kOk;
   const Terms terms = pack_terms(t0, p0, s0, z0, c0, t1, p1, s1, z1, c1, t2, p2, s2, z2, c2, t3, p3, s3, z3, c3);
-  if (dtype == TIE_F32) return launch_add_layer_norm<float>(x, terms, rows, w, bias, eps, out, n, D, s);
-  if (dtype == TIE_BF16) return launch_add_layer_norm<__nv_bfloat16>(x, terms, rows, w, bias, eps, out, n, D, s);
+  if (dtype == TIE_F32) return launch_add_layer_norm<float, true>(x, terms, rows, w, bias, eps, out, n, D, s);
+  if (dtype == TIE_BF16) return launch_add_layer_norm<__nv_bfloat16, true>(x, terms, rows, w, bias, eps, out, n, D, s);
+  set_error("unknown dtype code %d", dtype);
+  return kBadArgument;
+}
+
+TIE_API int tie_add_terms_rmsnorm(int dtype, float* x, TIE_TERMS, const int* rows, const float* w, float eps, void* out, int n, int D,
+                                  cudaStream_t s) {
+  TIE_REQUIRE(n >= 0 && D > 0, "add_terms_rmsnorm: bad sizes n=%d D=%d", n, D);
+  if (n == 0) return kOk;
+  const Terms terms = pack_terms(t0, p0, s0, z0, c0, t1, p1, s1, z1, c1, t2, p2, s2, z2, c2, t3, p3, s3, z3, c3);
+  if (dtype == TIE_F32) return launch_add_layer_norm<float, false>(x, terms, rows, w, nullptr, eps, out, n, D, s);
+  if (dtype == TIE_BF16) return launch_add_layer_norm<__nv_bfloat16, false>(x, terms, rows, w, nullptr, eps, out, n, D, s);
   set_error("unknown dtype code %d", dtype);
   return kBadArgument;
 }

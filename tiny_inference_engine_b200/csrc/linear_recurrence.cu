@@ -11,6 +11,7 @@
 // Kernels (float inside; T is the storage type of the projections and of the outputs that feed a product):
 //   gla_prep      one block per token.
 //   act_split     q, k, v behind an activation as float rows (linear attention with constant decays).
+//   rope_split    q and k rotated, k times a factor, and v, as float rows (one block per token; a token's angles are formed once).
 //   ssd_prep      one block per (token, unit): units are the heads of C, of B and of x, and one for the step sizes.
 //                 The convolution's first taps - 1 inputs come from the rows ahead in the step or from the tail that
 //                 the sequence's state slot keeps behind S (channels in the order C, B, x).
@@ -18,7 +19,7 @@
 //   ssd_out       one block per (token, part of the row).
 #include <math.h>
 
-#include "common.cuh"
+#include "rotation.cuh"
 
 namespace tie {
 
@@ -88,6 +89,84 @@ __global__ void __launch_bounds__(256) act_split_vec_kernel(const T* __restrict_
   }
 }
 
+// One block per token: cos and sin of the token's angles into shared memory, then q and k heads with their first turn.rot
+// dimensions rotated (k times k_scale) and v, as float rows. Heads' columns in pieces of four where everything is aligned.
+template <typename T>
+__global__ void __launch_bounds__(256) rope_split_kernel(const T* __restrict__ proj, long long stride, int q_off, int k_off, int v_off,
+                                                         int heads, int dim, int nv, Rotation turn, const int* __restrict__ positions,
+                                                         float k_scale, float* __restrict__ qn, float* __restrict__ kn,
+                                                         float* __restrict__ vn, int wide) {
+  pdl_sync();
+  extern __shared__ float cs[];              // [rot / 2] cosines, [rot / 2] sines
+  const long long t = blockIdx.x;
+  const int half = turn.rot / 2, nqk = heads * dim;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) turn.angle(positions[t], i, cs[i], cs[half + i]);
+  __syncthreads();
+  const T* row = proj + t * stride;
+  float* qd = qn + t * nqk;
+  float* kd = kn + t * nqk;
+  if (wide) {                                // dim, nv and (halves) rot / 2 or (neighbours) rot in pieces of four
+    const int per = dim / 4, items = 2 * heads * per;
+    for (int it = threadIdx.x; it < items; it += blockDim.x) {
+      const bool is_k = it >= heads * per;
+      const int in = is_k ? it - heads * per : it, h = in / per, d = (in % per) * 4;
+      const T* src = row + (is_k ? k_off : q_off) + h * dim;
+      float* dst = (is_k ? kd : qd) + h * dim;
+      const float c = is_k ? k_scale : 1.0f;
+      float u[4];
+      load4(src + d, u);
+      if (d >= turn.rot) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) u[e] *= c;
+        store4(dst + d, u);
+      } else if (turn.neighbours) {
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const float cc = cs[(d + e) / 2], ss = cs[half + (d + e) / 2], a = u[e], b = u[e + 1];
+          u[e] = c * (a * cc - b * ss);
+          u[e + 1] = c * (b * cc + a * ss);
+        }
+        store4(dst + d, u);
+      } else if (d < half) {                 // this thread makes both members of its four pairs
+        float v[4], a[4], b[4];
+        load4(src + d + half, v);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float cc = cs[d + e], ss = cs[half + d + e];
+          a[e] = c * (u[e] * cc - v[e] * ss);
+          b[e] = c * (v[e] * cc + u[e] * ss);
+        }
+        store4(dst + d, a);
+        store4(dst + d + half, b);
+      }
+    }
+    for (int d = threadIdx.x * 4; d < nv; d += blockDim.x * 4) {
+      float u[4];
+      load4(row + v_off + d, u);
+      store4(vn + t * nv + d, u);
+    }
+    return;
+  }
+  const int rest = dim - turn.rot, per = half + rest;      // pairs, then the dimensions that pass
+  for (int it = threadIdx.x; it < 2 * heads * per; it += blockDim.x) {
+    const bool is_k = it >= heads * per;
+    const int in = is_k ? it - heads * per : it, h = in / per, i = in % per;
+    const T* src = row + (is_k ? k_off : q_off) + h * dim;
+    float* dst = (is_k ? kd : qd) + h * dim;
+    const float c = is_k ? k_scale : 1.0f;
+    if (i < half) {
+      const int j1 = turn.first(i), j2 = turn.second(i);
+      const float a = ld(src + j1), b = ld(src + j2), cc = cs[i], ss = cs[half + i];
+      dst[j1] = c * (a * cc - b * ss);
+      dst[j2] = c * (b * cc + a * ss);
+    } else {
+      const int d = turn.rot + i - half;
+      dst[d] = c * ld(src + d);
+    }
+  }
+  for (int d = threadIdx.x; d < nv; d += blockDim.x) vn[t * nv + d] = ld(row + v_off + d);
+}
+
 struct SsdShape {
   int heads, groups, state, vdim, taps;
 };
@@ -142,7 +221,8 @@ __global__ void __launch_bounds__(128) ssd_prep_kernel(const T* __restrict__ pro
   }
 }
 
-// out[t, h] = (o[t, h] / rms(o[t, h])) * w * act(gate[t, h]); act 0: sigmoid, 1: silu. The gate has the storage type.
+// out[t, h] = (o[t, h] / rms(o[t, h])) * w * act(gate[t, h]) (w null: no weight); act 0: sigmoid, 1: silu. The gate has the
+// storage type.
 template <typename T>
 __global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate,
                                                              long long gate_stride, const float* __restrict__ w, float eps,
@@ -162,7 +242,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* __rest
   for (int d = lane; d < vdim; d += 32) {
     const float g = ld(gate + t * gate_stride + h * vdim + d);
     const float a = act == 1 ? g * lr_sigmoid(g) : lr_sigmoid(g);
-    st(out + item * vdim + d, ((x[d] * inv) * w[d]) * a);
+    st(out + item * vdim + d, (w != nullptr ? (x[d] * inv) * w[d] : x[d] * inv) * a);
   }
 }
 
@@ -182,7 +262,7 @@ __global__ void __launch_bounds__(256) head_norm_gate_block_kernel(const float* 
   for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
     const float g = ld(gate + t * gate_stride + h * vdim + d);
     const float a = act == 1 ? g * lr_sigmoid(g) : lr_sigmoid(g);
-    st(out + item * vdim + d, ((x[d] * inv) * w[d]) * a);
+    st(out + item * vdim + d, (w != nullptr ? (x[d] * inv) * w[d] : x[d] * inv) * a);
   }
 }
 
@@ -211,8 +291,8 @@ __global__ void __launch_bounds__(1024) head_norm_gate_vec4_kernel(const float* 
   for (int i = 0; i < NV; ++i) {
     const int d = (threadIdx.x + i * blockDim.x) * 4;
     if (d < vdim) {
-      float ww[4], r[4];
-      load4(w + d, ww);
+      float ww[4] = {1.0f, 1.0f, 1.0f, 1.0f}, r[4];
+      if (w != nullptr) load4(w + d, ww);
 #pragma unroll
       for (int e = 0; e < 4; ++e) r[e] = ((x[i][e] * inv) * ww[e]) * (act == 1 ? gv[i][e] * lr_sigmoid(gv[i][e]) : lr_sigmoid(gv[i][e]));
       store4(out + item * vdim + d, r);
@@ -294,6 +374,23 @@ TIE_API int tie_act_split(int dtype, const void* proj, long long stride, int q_o
                                    nv, act, qn, kn, vn, total));
   }
   TIE_RETURN_LAUNCH("act_split");
+}
+
+TIE_API int tie_rope_split(int dtype, const void* proj, long long stride, int q_off, int k_off, int v_off, int tokens, int heads, int dim,
+                           int nv, const float* inv_freq, const double* turns, int rot, int neighbours, const int* positions,
+                           float k_scale, float* qn, float* kn, float* vn, cudaStream_t s) {
+  TIE_REQUIRE(heads > 0 && dim > 0 && nv > 0 && rot >= 0 && rot % 2 == 0 && rot <= dim, "rope_split: bad sizes heads=%d dim=%d rot=%d nv=%d",
+              heads, dim, rot, nv);
+  TIE_REQUIRE(rot == 0 || ((inv_freq == nullptr) != (turns == nullptr) && positions != nullptr), "rope_split: a rotation takes one table of frequencies");
+  TIE_REQUIRE(rot <= 8192, "rope_split: %d rotated dimensions", rot);
+  if (tokens <= 0) return kOk;
+  auto on16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const bool wide = on16(proj) && on16(qn) && on16(kn) && on16(vn) && stride % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && v_off % 4 == 0 &&
+                    dim % 4 == 0 && nv % 4 == 0 && (neighbours ? rot % 4 == 0 : rot % 8 == 0);
+  const Rotation turn{inv_freq, turns, rot, neighbours};
+  TIE_BY_DTYPE(dtype, TIE_LAUNCH((rope_split_kernel<T>), tokens, 256, rot * sizeof(float), s, static_cast<const T*>(proj), stride, q_off, k_off,
+                                 v_off, heads, dim, nv, turn, positions, k_scale, qn, kn, vn, wide ? 1 : 0));
+  TIE_RETURN_LAUNCH("rope_split");
 }
 
 TIE_API int tie_ssd_prep(int dtype, const void* proj, long long stride, int c_off, int b_off, int x_off, int dt_off,

@@ -158,14 +158,25 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
     call("tie_silu_mul", dtype_code(out), gate_up.data_ptr(), out.data_ptr(), T, I, _stream())
 
 
-def rope(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, heads: int, head_dim: int) -> None:
-    """Rotate-half RoPE in place over the first 2*len(inv_freq) dims of each head of x [T, >= heads*head_dim]."""
-    _dev(x, positions, inv_freq)
+def _rotation(table, neighbours, what: str) -> tuple:
+    """A rotation's arguments of a launcher: (float32 inverse frequencies, float64 turns a position, pairing); `table` is one of
+    the two, or None."""
+    _dev(table)
+    if table is None:
+        return 0, 0, 0
+    _need(table.dtype in (torch.float32, torch.float64) and table.is_contiguous(), f"{what}: a rotation's table must be float32 inverse frequencies or float64 turns")
+    return (table.data_ptr(), 0, int(bool(neighbours))) if table.dtype == torch.float32 else (0, table.data_ptr(), int(bool(neighbours)))
+
+
+def rope(x: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, heads: int, head_dim: int, neighbours: bool = False) -> None:
+    """RoPE in place over the first 2*len(table) dims of each head of x [T, >= heads*head_dim]: dimension i with i + len(table), or
+    2i with 2i + 1 (`neighbours`). `table`: float32 inverse frequencies (angles are float products), or float64 turns a position
+    (angles formed in double)."""
+    _dev(x, positions)
     _need(x.dim() == 2 and x.stride(1) == 1 and x.shape[1] >= heads * head_dim, "rope: x must be [T, heads*head_dim]")
     _need(positions.dtype == torch.int32 and positions.numel() == x.shape[0], "rope: positions must be int32 [T]")
-    _need(inv_freq.dtype == torch.float32, "rope: inv_freq must be float32")
-    call("tie_rope", dtype_code(x), x.data_ptr(), x.stride(0), positions.data_ptr(), inv_freq.data_ptr(), x.shape[0],
-         heads, head_dim, 2 * inv_freq.numel(), _stream())
+    call("tie_rope", dtype_code(x), x.data_ptr(), x.stride(0), positions.data_ptr(), *_rotation(table, neighbours, "rope"), x.shape[0],
+         heads, head_dim, 2 * table.numel(), _stream())
 
 
 def _check_planes(k_cache, v_cache, kv_heads, head_dim):
@@ -313,7 +324,7 @@ def attention_decode_tc(q, k_cache, v_cache, out, query_start, context_lens, blo
          head_dim, k_cache.shape[2], int(window), float(scale), seq_list.data_ptr(), n_list, split_keys, max_splits,
          scratch.data_ptr(), _stream())
     call("tie_attention_merge", dtype_code(out), out.data_ptr(), query_start.data_ptr(), context_lens.data_ptr(), q_heads,
-         head_dim, int(window), seq_list.data_ptr(), n_list, split_keys, max_splits, scratch.data_ptr(), _stream())
+         head_dim, int(window), seq_list.data_ptr(), n_list, split_keys, max_splits, scratch.data_ptr(), 0, _stream())
 
 
 def attention_decode_tma_takes(q: torch.Tensor, q_heads: int, kv_heads: int, head_dim: int, page_size: int) -> bool:
@@ -477,7 +488,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, partial_scratch=No
 
 def bound_gemm(w: torch.Tensor, silu=False, split_many: bool = True, pack: bool = True):
     """A matrix product bound to one weight (gemm_select.BoundGemm): checked once, called every step.
-    `silu`: the epilogue of a gated unit, True or GATED_SILU: silu(gate) * up, GATED_RELU: max(gate, 0) * up.
+    `silu`: an epilogue. Of a gated unit, True or GATED_SILU: silu(gate) * up, GATED_RELU: max(gate, 0) * up; SQUARED_RELU: max(., 0)^2.
     `split_many` False: above 128 tokens k is never split (the consumer wants the finished product). With `pack`
     a weight that the tensor-core kernels take is stored in k-blocks (pack_k_blocks) from here on: the product
     keeps that copy (`.w`) and the caller lets go of its own. `.rows(a, b)` is the product with rows a..b-1 of
@@ -552,7 +563,8 @@ def glu_clamped(gate_up: torch.Tensor, out: torch.Tensor, limit: float, slope: f
          float(up_shift), _stream())
 
 
-GATED_SILU, GATED_RELU = 1, 2      # the epilogues of a gated product
+# The epilogues of a product: 1, 2 act(gate) * up of a gated unit; 3 max(product, 0)^2.
+GATED_SILU, GATED_RELU, SQUARED_RELU = 1, 2, 3
 
 
 def sigmoid_gate_mul(y: torch.Tensor, gate: torch.Tensor) -> None:
@@ -582,22 +594,22 @@ def _check_kv_planes(k_cache, v_cache, kv_heads, head_dim, v_dim):
     _need(max(k_cache.numel() // head_dim, v_cache.numel() // v_cache.shape[3]) < 2 ** 31, "cache plane too large for 32-bit row indices")
 
 
-def qkv_span_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bq, bk, bv, wq, wk, eps: float, inv_freq,
+def qkv_span_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bq, bk, bv, wq, wk, eps: float, table,
                   positions: torch.Tensor, slots, k_cache, v_cache, q_heads: int, kv_heads: int, head_dim: int, v_dim: int,
-                  mix_mode: int = 0, v_first=None, mix_weight=None, write_kv: bool = True) -> None:
+                  mix_mode: int = 0, v_first=None, mix_weight=None, write_kv: bool = True, neighbours: bool = False) -> None:
     """proj [T, >= ...] holds the q, k and v projections of every token at columns q_off, k_off, v_off. q gets its
     bias, the RMS norm over all of its heads at once (weights wq, float32 [q_heads * head_dim]) and the rotation of
-    the first 2 * len(inv_freq) dimensions of each head, and is written back in place; k likewise into the key
+    the first 2 * len(table) dimensions of each head (`table`, `neighbours` as for `rope`; None: no rotation), and is written back in place; k likewise into the key
     plane; v gets its bias, is kept as `v_first` (mix_mode 1) or blended with it, (1 - w) v + w v_first (mix_mode 2,
     `mix_weight` a float32 device scalar), and goes into the value plane."""
-    _dev(proj, bq, bk, bv, wq, wk, inv_freq, positions, slots, k_cache, v_cache, v_first, mix_weight)
+    _dev(proj, bq, bk, bv, wq, wk, positions, slots, k_cache, v_cache, v_first, mix_weight)
     T = proj.shape[0]
     nq, nk, nv = q_heads * head_dim, kv_heads * head_dim, kv_heads * v_dim
     _need(proj.dim() == 2 and proj.stride(1) == 1 and q_off + nq <= proj.shape[1], "qkv_span_prep: q outside the projection")
     _need(positions.dtype == torch.int32 and positions.numel() == T, "qkv_span_prep: positions must be int32 [T]")
     for t, n in ((bq, nq), (bk, nk), (bv, nv), (wq, nq), (wk, nk)):
         _need(t is None or (t.dtype == torch.float32 and t.numel() == n), "qkv_span_prep: biases and norm weights must be float32 of the projection's size")
-    _need(inv_freq is None or inv_freq.dtype == torch.float32, "qkv_span_prep: inv_freq must be float32")
+    inv_freq, turns, pairing = _rotation(table, neighbours, "qkv_span_prep")
     page = 1
     if write_kv:
         _need(max(k_off + nk, v_off + nv) <= proj.shape[1], "qkv_span_prep: k or v outside the projection")
@@ -612,11 +624,17 @@ def qkv_span_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bq, bk
             _need(mix_mode == 1 or (mix_weight is not None and mix_weight.dtype == torch.float32 and mix_weight.numel() == 1),
                   "qkv_span_prep: the blend's weight must be a float32 scalar on the device")
     call("tie_qkv_span_prep", dtype_code(proj), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, _ptr(bq), _ptr(bk), _ptr(bv),
-         _ptr(wq), _ptr(wk), float(eps), _ptr(inv_freq), 2 * inv_freq.numel() if inv_freq is not None else 0,
+         _ptr(wq), _ptr(wk), float(eps), inv_freq, turns, 2 * table.numel() if table is not None else 0, pairing,
          positions.data_ptr(), _ptr(slots) if write_kv else 0, _ptr(k_cache) if write_kv else 0,
          _ptr(v_cache) if write_kv else 0, T, q_heads, kv_heads, head_dim, v_dim, v_cache.shape[3] if write_kv else v_dim, page,
          int(mix_mode) if write_kv else 0,
          _ptr(v_first), _ptr(mix_weight), _stream())
+
+
+def _sink_ptr(sink, q_heads: int) -> int:
+    _dev(sink)
+    _need(sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == q_heads), "attention: sinks must be float32 [q_heads]")
+    return _ptr(sink)
 
 
 def _attn_common_dv(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim,
@@ -639,9 +657,10 @@ def _attn_common_dv(q, k_cache, v_cache, out, query_start, context_lens, block_t
 
 
 def attention_rows_dv(q, k_cache, v_cache, out, seq_of_row, query_start, context_lens, block_tables, q_heads, kv_heads,
-                      head_dim, v_dim, scale: float, window: int = 0, values_in_keys: bool = False) -> None:
+                      head_dim, v_dim, scale: float, window: int = 0, values_in_keys: bool = False, sink=None) -> None:
     """`attention_rows` for keys of head_dim and values of v_dim (out [T, q_heads * v_dim]). `values_in_keys`: there
-    is no value plane; a value is the first v_dim elements of its key (pass the key plane as `v_cache`)."""
+    is no value plane; a value is the first v_dim elements of its key (pass the key plane as `v_cache`). `sink` (float32
+    [q_heads] or None): exp(sink[h]) is one more term of head h's softmax denominator."""
     _dev(q, k_cache, v_cache, out, seq_of_row, query_start, context_lens, block_tables)
     S = _attn_common_dv(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim,
                         values_in_keys)
@@ -649,14 +668,14 @@ def attention_rows_dv(q, k_cache, v_cache, out, seq_of_row, query_start, context
     call("tie_attention_rows_dv", dtype_code(q), q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
          out.data_ptr(), seq_of_row.data_ptr(), query_start.data_ptr(), context_lens.data_ptr(), block_tables.data_ptr(),
          block_tables.shape[1], q.shape[0], S, q_heads, kv_heads, head_dim, v_dim, k_cache.shape[2], int(window), float(scale),
-         head_dim if values_in_keys else 0, _stream())
+         head_dim if values_in_keys else 0, _sink_ptr(sink, q_heads), _stream())
 
 
 def attention_split_dv(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim,
                        scale: float, seq_list, n_list: int, split_keys: int, max_splits: int, scratch, window: int = 0,
-                       values_in_keys: bool = False) -> None:
+                       values_in_keys: bool = False, sink=None) -> None:
     """`attention_split` for keys of head_dim and values of v_dim; scratch holds
-    attention_split_scratch_floats(n_list, q_heads, v_dim, max_splits) floats. `values_in_keys` as in `attention_rows_dv`."""
+    attention_split_scratch_floats(n_list, q_heads, v_dim, max_splits) floats. `values_in_keys` and `sink` as in `attention_rows_dv`."""
     _dev(q, k_cache, v_cache, out, query_start, context_lens, block_tables, seq_list, scratch)
     S = _attn_common_dv(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim,
                         values_in_keys)
@@ -666,7 +685,7 @@ def attention_split_dv(q, k_cache, v_cache, out, query_start, context_lens, bloc
     call("tie_attention_split_dv", dtype_code(q), q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
          out.data_ptr(), query_start.data_ptr(), context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1],
          S, q_heads, kv_heads, head_dim, v_dim, k_cache.shape[2], int(window), float(scale), seq_list.data_ptr(), n_list,
-         split_keys, max_splits, scratch.data_ptr(), head_dim if values_in_keys else 0, _stream())
+         split_keys, max_splits, scratch.data_ptr(), head_dim if values_in_keys else 0, _sink_ptr(sink, q_heads), _stream())
 
 
 # -- the gated delta rule with a decay per key channel (csrc/delta_rule.cu)
@@ -797,16 +816,16 @@ GATE_SIGMOID, GATE_SILU = 0, 1
 
 
 def head_norm_gate(o, gate, weight, eps: float, out, heads: int, vdim: int, act: int = GATE_SIGMOID) -> None:
-    """out[t, h] = (o[t, h] / rms(o[t, h])) * weight * act(gate[t, h]) per head of vdim; o float32, gate (rows may be
-    strided) and out in the compute dtype; act GATE_SIGMOID or GATE_SILU."""
+    """out[t, h] = (o[t, h] / rms(o[t, h])) * weight * act(gate[t, h]) per head of vdim (weight float32 [vdim], or None for 1); o
+    float32, gate (rows may be strided) and out in the compute dtype; act GATE_SIGMOID or GATE_SILU."""
     _dev(o, gate, weight, out)
     T = o.shape[0]
     _need(o.dtype == torch.float32 and o.is_contiguous() and o.shape == (T, heads * vdim), "head_norm_gate: o must be float32 [T, heads * vdim]")
     _need(gate.dim() == 2 and gate.stride(1) == 1 and gate.shape == o.shape and gate.dtype == out.dtype,
           "head_norm_gate: gate must be [T, heads * vdim] in out's dtype")
-    _need(weight.dtype == torch.float32 and weight.numel() == vdim, "head_norm_gate: weight must be float32 [vdim]")
+    _need(weight is None or (weight.dtype == torch.float32 and weight.numel() == vdim), "head_norm_gate: weight must be float32 [vdim]")
     _need(out.is_contiguous() and out.shape == o.shape, "head_norm_gate: out must be [T, heads * vdim] contiguous")
-    call("tie_head_norm_gate", dtype_code(out), o.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), float(eps),
+    call("tie_head_norm_gate", dtype_code(out), o.data_ptr(), gate.data_ptr(), gate.stride(0), _ptr(weight), float(eps),
          out.data_ptr(), T, heads, vdim, int(act), _stream())
 
 
@@ -828,38 +847,37 @@ def ssd_out(o, xn, z, skip, weight, eps: float, out, heads: int, vdim: int, part
 
 # -- attention over one latent per token (csrc/attention_latent.cu) and products batched over heads
 
-def latent_prep(proj, q_off: int, q_rank: int, kv_off: int, rank: int, rot: int, wq, wkv, eps: float, inv_freq, positions,
-                slots, cq, k_cache) -> None:
+def latent_prep(proj, q_off: int, q_rank: int, kv_off: int, rank: int, rot: int, wq, wkv, eps: float, table, positions,
+                slots, cq, k_cache, neighbours: bool = False) -> None:
     """From the stacked down-projections of every token: cq [T, q_rank] = rmsnorm(proj[q_off:]) * wq; the key plane's row
-    at the token's slot = [rmsnorm(proj[kv_off : kv_off + rank]) * wkv | rotation of the `rot` columns behind them]."""
-    _dev(proj, wq, wkv, inv_freq, positions, slots, cq, k_cache)
+    at the token's slot = [rmsnorm(proj[kv_off : kv_off + rank]) * wkv | rotation of the `rot` columns behind them] (`table`,
+    `neighbours` as for `rope`)."""
+    _dev(proj, wq, wkv, positions, slots, cq, k_cache)
     T = proj.shape[0]
     _need(proj.dim() == 2 and proj.stride(1) == 1 and max(q_off + q_rank, kv_off + rank + rot) <= proj.shape[1],
           "latent_prep: columns outside the projection")
     _need(wq.dtype == torch.float32 and wq.numel() == q_rank and wkv.dtype == torch.float32 and wkv.numel() == rank,
           "latent_prep: norm weights must be float32 of the latents' sizes")
-    _need(rot == 0 or (inv_freq is not None and inv_freq.dtype == torch.float32 and 2 * inv_freq.numel() == rot),
-          "latent_prep: inv_freq must be float32 [rot / 2]")
+    _need(rot == 0 or (table is not None and 2 * table.numel() == rot), "latent_prep: a table of [rot / 2] frequencies")
     _need(positions.dtype == torch.int32 and positions.numel() == T and slots.dtype == torch.int32 and slots.numel() == T,
           "latent_prep: positions and slots must be int32 [T]")
     _need(cq.shape == (T, q_rank) and cq.is_contiguous() and cq.dtype == proj.dtype, "latent_prep: cq must be [T, q_rank] contiguous")
     _need(k_cache.dim() == 4 and k_cache.is_contiguous() and k_cache.shape[1] == 1 and k_cache.shape[3] == rank + rot and
           k_cache.dtype == proj.dtype, "latent_prep: the key plane must be [pages, 1, page_size, rank + rot]")
     call("tie_latent_prep", dtype_code(proj), proj.data_ptr(), proj.stride(0), q_off, q_rank, kv_off, rank, rot, wq.data_ptr(),
-         wkv.data_ptr(), float(eps), _ptr(inv_freq), positions.data_ptr(), slots.data_ptr(), cq.data_ptr(), k_cache.data_ptr(),
+         wkv.data_ptr(), float(eps), *_rotation(table if rot else None, neighbours, "latent_prep"), positions.data_ptr(), slots.data_ptr(), cq.data_ptr(), k_cache.data_ptr(),
          T, _stream())
 
 
-def latent_query_rot(q, dim: int, rot: int, inv_freq, positions, folded, rank: int, heads: int) -> None:
+def latent_query_rot(q, dim: int, rot: int, table, positions, folded, rank: int, heads: int, neighbours: bool = False) -> None:
     """folded[t, h, rank : rank + rot] = rotation of q[t, h, dim : dim + rot] (heads of dim + rot in q, of rank + rot in folded)."""
-    _dev(q, inv_freq, positions, folded)
+    _dev(q, positions, folded)
     T = q.shape[0]
     _need(q.dim() == 2 and q.stride(1) == 1 and q.shape[1] >= heads * (dim + rot) and folded.dim() == 2 and folded.stride(1) == 1
           and folded.shape == (T, heads * (rank + rot)) and folded.dtype == q.dtype, "latent_query_rot: q [T, heads * (dim + rot)], folded [T, heads * (rank + rot)]")
-    _need(rot == 0 or (inv_freq is not None and inv_freq.dtype == torch.float32 and 2 * inv_freq.numel() == rot),
-          "latent_query_rot: inv_freq must be float32 [rot / 2]")
+    _need(rot == 0 or (table is not None and 2 * table.numel() == rot), "latent_query_rot: a table of [rot / 2] frequencies")
     _need(positions.dtype == torch.int32 and positions.numel() == T, "latent_query_rot: positions must be int32 [T]")
-    call("tie_latent_query_rot", dtype_code(q), q.data_ptr(), q.stride(0), dim, rot, _ptr(inv_freq), positions.data_ptr(),
+    call("tie_latent_query_rot", dtype_code(q), q.data_ptr(), q.stride(0), dim, rot, *_rotation(table if rot else None, neighbours, "latent_query_rot"), positions.data_ptr(),
          folded.data_ptr(), folded.stride(0), rank, heads, T, _stream())
 
 
@@ -881,21 +899,22 @@ def _latent_common(q, k_cache, query_start, context_lens, block_tables, heads, k
 
 
 def attention_latent_prompt(q, k_cache, out, query_start, context_lens, block_tables, n_seqs: int, max_queries: int, heads: int,
-                            key_dim: int, rank: int, scale: float, window: int = 0) -> None:
+                            key_dim: int, rank: int, scale: float, window: int = 0, sink=None) -> None:
     """Attention of the first n_seqs sequences of the step (each brings several tokens; their rows come first) over a
     keys-only cache: every head reads the same rows of key_dim, a key's first `rank` elements are its value.
-    q [T, heads * key_dim], out [T, heads * rank], bfloat16, on the tensor cores; softmax in float."""
+    q [T, heads * key_dim], out [T, heads * rank], bfloat16, on the tensor cores; softmax in float. `sink` (float32 [heads] or
+    None): exp(sink[h]) is one more term of head h's softmax denominator."""
     _dev(q, k_cache, out, query_start, context_lens, block_tables)
     _latent_common(q, k_cache, query_start, context_lens, block_tables, heads, key_dim, rank)
     _need(out.shape == (q.shape[0], heads * rank) and out.is_contiguous() and out.dtype == torch.bfloat16,
           "latent attention: out must be bfloat16 [T, heads * rank] contiguous")
     call("tie_attention_latent_prompt", q.data_ptr(), q.stride(0), k_cache.data_ptr(), out.data_ptr(), query_start.data_ptr(),
          context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], n_seqs, max_queries, heads, key_dim, rank,
-         k_cache.shape[2], int(window), float(scale), _stream())
+         k_cache.shape[2], int(window), float(scale), _sink_ptr(sink, heads), _stream())
 
 
 def attention_latent_split(q, k_cache, out, query_start, context_lens, block_tables, heads: int, key_dim: int, rank: int,
-                           scale: float, seq_list, n_list: int, split_keys: int, max_splits: int, scratch, window: int = 0) -> None:
+                           scale: float, seq_list, n_list: int, split_keys: int, max_splits: int, scratch, window: int = 0, sink=None) -> None:
     """The same for sequences that bring one token each, their keys cut into splits of `split_keys` that are merged in
     split order; scratch holds attention_split_scratch_floats(n_list, heads, rank, max_splits) floats."""
     _dev(q, k_cache, out, query_start, context_lens, block_tables, seq_list, scratch)
@@ -909,7 +928,7 @@ def attention_latent_split(q, k_cache, out, query_start, context_lens, block_tab
          context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], heads, key_dim, rank, k_cache.shape[2],
          int(window), float(scale), seq_list.data_ptr(), n_list, split_keys, max_splits, scratch.data_ptr(), _stream())
     call("tie_attention_merge", dtype_code(out), out.data_ptr(), query_start.data_ptr(), context_lens.data_ptr(), heads, rank,
-         int(window), seq_list.data_ptr(), n_list, split_keys, max_splits, scratch.data_ptr(), _stream())
+         int(window), seq_list.data_ptr(), n_list, split_keys, max_splits, scratch.data_ptr(), _sink_ptr(sink, heads), _stream())
 
 
 def head_gate_mul(y, gate, heads: int, head_size: int) -> None:
@@ -1284,7 +1303,7 @@ def attention_mixed(q, k_cache, v_cache, out, mix, ctx_arrays, rows: int, heads:
          _ptr(seq_list) if split else 0, n_list, split_keys, max_splits, _ptr(scratch) if split else 0, _stream())
     if split and n_list > 0:
         call("tie_attention_merge", dtype_code(out), out.data_ptr(), query_start.data_ptr(), context_lens.data_ptr(), heads, vdim,
-             0, seq_list.data_ptr(), n_list, split_keys, max_splits, scratch.data_ptr(), _stream())
+             0, seq_list.data_ptr(), n_list, split_keys, max_splits, scratch.data_ptr(), 0, _stream())
 
 
 def attention_mixed_tc_takes(heads: int, kv_heads: int, dim: int, vdim: int) -> bool:
@@ -1314,7 +1333,7 @@ def attention_mixed_tc(q, k_cache, v_cache, out, mix, query_start, context_lens,
          _ptr(seq_list) if split else 0, int(split_keys), int(max_splits), _ptr(scratch) if split else 0, _stream())
     if split and n_seqs > 0:
         call("tie_attention_merge", dtype_code(out), out.data_ptr(), query_start.data_ptr(), context_lens.data_ptr(), heads, vdim,
-             0, seq_list.data_ptr(), n_seqs, split_keys, max_splits, scratch.data_ptr(), _stream())
+             0, seq_list.data_ptr(), n_seqs, split_keys, max_splits, scratch.data_ptr(), 0, _stream())
 
 
 # -- a norm without statistics and a sinusoid on the embedding (csrc/tanh_norm.cu)
@@ -1375,6 +1394,13 @@ def sinusoid_add(x: torch.Tensor, positions: torch.Tensor, base: float = 10000.0
     _need(x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2, "sinusoid_add: x must be float32 [T, D] contiguous")
     _need(positions.dtype == torch.int32 and positions.numel() >= x.shape[0], "sinusoid_add: positions must be int32 [T]")
     call("tie_sinusoid_add", x.data_ptr(), positions.data_ptr(), x.shape[0], x.shape[1], float(base), _stream())
+
+
+def squared_relu(z: torch.Tensor, out: torch.Tensor) -> None:
+    """out = max(z, 0)^2; z and out alike, contiguous (out may be z)."""
+    _dev(z, out)
+    _need(z.shape == out.shape and z.dtype == out.dtype and z.is_contiguous() and out.is_contiguous(), "squared_relu: z and out alike, contiguous")
+    call("tie_squared_relu", dtype_code(z), z.data_ptr(), out.data_ptr(), z.numel(), _stream())
 
 
 def two_branch_unit(z: torch.Tensor, out: torch.Tensor, c_pos: float, c_neg: float) -> None:
@@ -1603,6 +1629,19 @@ def add_layer_norm(x, delta, weight, bias, eps: float, out, rows=None) -> None:
          weight.data_ptr(), bias.data_ptr(), float(eps), out.data_ptr(), n, D, _stream())
 
 
+def add_terms_rmsnorm(x, delta, weight, eps: float, out, rows=None) -> None:
+    """x += delta (float32, in place; as for `add_layer_norm`), out = x / sqrt(mean(x^2) + eps) * weight in out's dtype."""
+    _dev(x, weight, out, rows)
+    D, n = x.shape[-1], out.shape[0]
+    _need(x.dtype == torch.float32 and x.is_contiguous(), "add_terms_rmsnorm: x must be float32 contiguous")
+    _need(weight.dtype == torch.float32 and weight.numel() == D, "add_terms_rmsnorm: weight must be float32 [D]")
+    _need(out.shape[-1] == D and out.is_contiguous(), "add_terms_rmsnorm: out must be [n, D] contiguous")
+    _need(rows is None and n == x.shape[0] or rows is not None and rows.dtype == torch.int32 and rows.numel() == n,
+          "add_terms_rmsnorm: out must have x's rows, or rows must be int32 [n]")
+    call("tie_add_terms_rmsnorm", dtype_code(out), x.data_ptr(), *_term_args(delta, x, out.dtype, "add_terms_rmsnorm"), _ptr(rows),
+         weight.data_ptr(), float(eps), out.data_ptr(), n, D, _stream())
+
+
 def stream_add(x, delta, dtype, other=None, vec=None) -> None:
     """x += delta (as for `add_layer_norm`; tensors of `dtype`), then += other (float32 rows), then += vec (float32 [D], every row)."""
     _dev(x, other, vec)
@@ -1717,13 +1756,23 @@ def act_split(proj, q_off: int, k_off: int, v_off: int, qn, kn, vn, silu: bool =
          kn.data_ptr(), vn.data_ptr(), _stream())
 
 
+def rope_split(proj, q_off: int, k_off: int, v_off: int, heads: int, dim: int, table, positions, k_scale: float, qn, kn, vn,
+               neighbours: bool = False) -> None:
+    """The q and k columns of `proj` (heads * dim each) with the first 2 * len(table) dimensions of each head rotated (`table`,
+    `neighbours` as for `rope`; None: no rotation), k times k_scale, and the v columns, as float32 rows qn, kn [T, heads * dim], vn."""
+    _dev(proj, positions, qn, kn, vn)
+    T, nqk, nv = proj.shape[0], heads * dim, vn.shape[1]
+    _need(proj.dim() == 2 and proj.stride(1) == 1 and max(q_off + nqk, k_off + nqk, v_off + nv) <= proj.shape[1], "rope_split: columns outside the projection")
+    for t, n in ((qn, nqk), (kn, nqk), (vn, nv)):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n), "rope_split: outputs must be float32 [T, n]")
+    _need(positions.dtype == torch.int32 and positions.numel() == T, "rope_split: positions must be int32 [T]")
+    inv_freq, turns, pairing = _rotation(table, neighbours, "rope_split")
+    call("tie_rope_split", dtype_code(proj), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, T, heads, dim, nv, inv_freq, turns,
+         2 * table.numel() if table is not None else 0, pairing, positions.data_ptr(), float(k_scale), qn.data_ptr(), kn.data_ptr(),
+         vn.data_ptr(), _stream())
+
+
 # -- attention in a window beside which the first keys stay visible, with capped scores and a sink per head
-
-def _kept_sink(sink, q_heads):
-    _dev(sink)
-    _need(sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == q_heads), "attention: sinks must be float32 [q_heads]")
-    return _ptr(sink)
-
 
 def attention_kept_rows(q, k_cache, v_cache, out, seq_of_row, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim,
                         scale: float, window: int = 0, keep_first: int = 0, softcap: float = 0.0, sink=None) -> None:
@@ -1735,7 +1784,7 @@ def attention_kept_rows(q, k_cache, v_cache, out, seq_of_row, query_start, conte
     call("tie_attention_kept_rows", dtype_code(q), q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
          seq_of_row.data_ptr(), query_start.data_ptr(), context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], q.shape[0], S,
          q_heads, kv_heads, head_dim, v_dim, k_cache.shape[2], int(window), int(keep_first), float(scale), float(softcap),
-         _kept_sink(sink, q_heads), _stream())
+         _sink_ptr(sink, q_heads), _stream())
 
 
 def attention_kept_split(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, v_dim, scale: float,
@@ -1749,7 +1798,7 @@ def attention_kept_split(q, k_cache, v_cache, out, query_start, context_lens, bl
           scratch.numel() >= attention_split_scratch_floats(n_list, q_heads, v_dim, max_splits), "attention: scratch too small")
     call("tie_attention_kept_split", dtype_code(q), q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
          query_start.data_ptr(), context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], S, q_heads, kv_heads, head_dim, v_dim,
-         k_cache.shape[2], int(window), int(keep_first), float(scale), float(softcap), _kept_sink(sink, q_heads), seq_list.data_ptr(), n_list,
+         k_cache.shape[2], int(window), int(keep_first), float(scale), float(softcap), _sink_ptr(sink, q_heads), seq_list.data_ptr(), n_list,
          split_keys, max_splits, scratch.data_ptr(), _stream())
 
 
@@ -1760,7 +1809,7 @@ def attention_prompt_kept(q, k_cache, v_cache, out, query_start, context_lens, b
     _attn_common(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim)
     call("tie_attention_prompt_kept", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), query_start.data_ptr(),
          context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], n_seqs, max_queries, q_heads, kv_heads, head_dim,
-         k_cache.shape[2], k_cache.shape[0], int(window), int(keep_first), float(scale), float(softcap), _kept_sink(sink, q_heads), _stream())
+         k_cache.shape[2], k_cache.shape[0], int(window), int(keep_first), float(scale), float(softcap), _sink_ptr(sink, q_heads), _stream())
 
 
 def attention_decode_kept(q, k_cache, v_cache, out, query_start, context_lens, block_tables, q_heads, kv_heads, head_dim, scale: float,
@@ -1776,5 +1825,5 @@ def attention_decode_kept(q, k_cache, v_cache, out, query_start, context_lens, b
     _need(counters.dtype == torch.int32 and counters.numel() >= n_list * kv_heads, "attention: counters too small")
     call("tie_attention_decode_kept", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), query_start.data_ptr(),
          context_lens.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], q_heads, kv_heads, head_dim, k_cache.shape[2],
-         k_cache.shape[0], int(window), int(keep_first), float(scale), float(softcap), _kept_sink(sink, q_heads), 0, first, n_list, split_keys,
+         k_cache.shape[0], int(window), int(keep_first), float(scale), float(softcap), _sink_ptr(sink, q_heads), 0, first, n_list, split_keys,
          max_splits, scratch.data_ptr(), counters.data_ptr(), 1 if cluster else 0, _stream())

@@ -156,6 +156,11 @@ def pair_width(M: int, N: int, K: int, pairs: int) -> int:
     return best[1]
 
 
+def _gated(epilogue) -> bool:
+    """Whether an epilogue is that of a gated unit (1, 2): the output is half as wide as the product, and k stays whole."""
+    return int(epilogue) in (1, 2)
+
+
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, transposed=None, bn=None, splits=None, scratch=None,
             silu=False, partial_scratch=None, deep=None, pair=None, checked: bool = False):
     """The tensor-core product; the tiling can be forced (tests). Returns `out`, or a SplitSum when
@@ -167,7 +172,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, transposed=None
     SplitSum, _need, _stream, dtype_code = _ops
     M, K = a.shape
     N = w.shape[0]
-    _need(w.shape[1] == K and out.shape == (M, N // 2 if silu else N),
+    _need(w.shape[1] == K and out.shape == (M, N // 2 if _gated(silu) else N),
           f"gemm: shapes {tuple(a.shape)} x {tuple(w.shape)}^T -> {tuple(out.shape)}")
     _need(a.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1, "gemm: last axes must be contiguous")
     _need(checked or tc_takes(a, w, out),
@@ -183,11 +188,11 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, transposed=None
     transposed = t if transposed is None else int(transposed)
     bn = b if bn is None else bn
     splits = s if splits is None else splits
-    if silu:
+    if _gated(silu):
         splits = 1
         if not transposed:
             bn = max(bn, 32)
-    leave = splits > 1 and partial_scratch is not None
+    leave = splits > 1 and partial_scratch is not None and not silu
     if leave:
         scratch = partial_scratch(splits * M * N)
     elif splits > 1 and scratch is None:
@@ -245,14 +250,15 @@ class BoundGemm:
     its rows (the q rows of a stacked q/k/v weight) over the same memory."""
 
     def __init__(self, w: torch.Tensor, silu=False, split_many: bool = True, pack: bool = True, _slice=None):
-        self.silu, self.split_many = int(silu), split_many      # 0: none, 1: the SiLU, 2: the ReLU of a gated unit
+        self.silu, self.split_many = int(silu), split_many      # 0: none, 1: the SiLU, 2: the ReLU of a gated unit, 3: the squared ReLU
+        self.gated = _gated(silu)
         if _slice is not None:              # rows [row0, row0 + N) of a packed weight
             parent, row0, n = _slice
             self.w, self.N, self.K, self.packed_rows, self.row0, self.fast = parent.w, n, parent.K, parent.packed_rows, row0, True
         else:
             self.N, self.K = w.shape
             self.fast = (w.dtype == torch.bfloat16 and w.stride(1) == 1 and self.K % 8 == 0 and w.stride(0) % 8 == 0
-                         and w.data_ptr() % 16 == 0 and (not silu or self.N % 32 == 0))
+                         and w.data_ptr() % 16 == 0 and (not self.gated or self.N % 32 == 0))
             self.packed_rows = self.row0 = 0
             if pack and self.fast and w.is_cuda:
                 from . import pack_k_blocks
@@ -280,7 +286,7 @@ class BoundGemm:
     def _plan(self, M: int):
         pair = pair_takes(M, self.N)
         t, bn, splits = plan(M, self.N, self.K, self.split_many)
-        if self.silu:
+        if self.gated:
             splits = 1
             if not t:
                 bn = max(bn, 32)
@@ -296,11 +302,16 @@ class BoundGemm:
         if M == 0:
             return out
         if not (self.fast and a.dtype == torch.bfloat16 and a.stride(1) == 1 and a.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0
-                and out.stride(1) == 1 and a.shape[1] == self.K and out.shape[1] == (self.N // 2 if self.silu else self.N)
+                and out.stride(1) == 1 and a.shape[1] == self.K and out.shape[1] == (self.N // 2 if self.gated else self.N)
                 and out.shape[0] == M and out.dtype in (torch.bfloat16, torch.float32)):
             w = self.row_major()
-            if self.silu:
+            if self.gated:
                 gemm_silu(a, w, out, self.silu)
+                return out
+            if self.silu:                   # the squared ReLU behind whichever product takes the operands
+                from . import squared_relu
+                gemm(a, w, out)
+                squared_relu(out, out)
                 return out
             return gemm(a, w, out, partial_scratch)
         global _ops
@@ -314,7 +325,7 @@ class BoundGemm:
             _call("tie_gemm_tc2", code, a.data_ptr(), self.w_ptr, out.data_ptr(), M, self.N, self.K, a.stride(0), self.ldw,
                   out.stride(0), self.silu, self.packed_rows, self.row0, bn, _stream())
             return out
-        leave = splits > 1 and partial_scratch is not None
+        leave = splits > 1 and partial_scratch is not None and not self.silu
         scratch = 0
         if leave:
             buf = partial_scratch(splits * M * self.N)

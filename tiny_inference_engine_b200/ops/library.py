@@ -22,7 +22,7 @@ _SIGNATURES = {
     "tie_add_rmsnorm": [I, P, P, P, L, I, P, P, F, P, I, I, P],
     "tie_rmsnorm_rows": [I, P, L, P, F, P, L, I, L, P],
     "tie_silu_mul": [I, P, P, I, I, P],
-    "tie_rope": [I, P, L, P, P, I, I, I, I, P],
+    "tie_rope": [I, P, L, P, P, P, I, I, I, I, I, P],
     "tie_kv_append": [I, P, P, L, L, P, P, P, I, I, I, I, P],
     "tie_qk_norm_rope_append": [I, P, L, P, L, I, L, P, P, F, F, P, I, P, P, P, P, I, I, I, I, I, I, P],
     "tie_gemm_simt": [I, I, P, P, P, I, I, I, L, L, L, P],
@@ -40,14 +40,14 @@ _SIGNATURES = {
     "tie_attention_prompt_tma": [P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P],
     "tie_attention_prompt_tma_exact": [P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P],
     "tie_attention_prompt_umma": [P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P],
-    "tie_attention_merge": [I, P, P, P, I, I, I, P, I, I, I, P, P],
-    "tie_attention_rows_dv": [I, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P],
-    "tie_attention_split_dv": [I, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, I, I, I, P, I, P],
+    "tie_attention_merge": [I, P, P, P, I, I, I, P, I, I, I, P, P, P],
+    "tie_attention_rows_dv": [I, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, P],
+    "tie_attention_split_dv": [I, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, I, I, I, P, I, P, P],
     "tie_add_normed_rmsnorm": [I, P, P, P, L, I, P, P, F, F, P, P, F, P, I, I, P],
     "tie_glu_clamped": [I, P, P, I, I, F, F, F, P],
     "tie_sigmoid_gate_mul": [I, P, L, P, L, I, I, P],
     "tie_scale_rows": [P, L, I, I, F, P],
-    "tie_qkv_span_prep": [I, P, L, I, I, I, P, P, P, P, P, F, P, I, P, P, P, P, I, I, I, I, I, I, I, I, P, P, P],
+    "tie_qkv_span_prep": [I, P, L, I, I, I, P, P, P, P, P, F, P, P, I, I, P, P, P, P, I, I, I, I, I, I, I, I, P, P, P],
     "tie_delta_prep": [I, P, L, I, I, I, I, P, P, L, L, P, P, P, I, I, I, I, I, I, F, F, P, P, P, P, P, L, P, P, P],
     "tie_delta_rule": [I, P, P, P, P, P, L, P, L, L, P, L, I, I, I, P, P, I, I, I, I, I, I, P, I, I, I, P],
     "tie_delta_out": [I, P, P, L, P, F, P, I, I, I, P],
@@ -56,10 +56,10 @@ _SIGNATURES = {
     "tie_ssd_prep": [I, P, L, I, I, I, I, P, P, P, L, L, P, P, P, I, I, I, I, I, I, P, P, P, P, P, P, P, P],
     "tie_head_norm_gate": [I, P, P, L, P, F, P, I, I, I, I, P],
     "tie_ssd_out": [I, P, P, P, L, P, P, F, P, I, I, I, I, P],
-    "tie_latent_prep": [I, P, L, I, I, I, I, I, P, P, F, P, P, P, P, P, I, P],
-    "tie_latent_query_rot": [I, P, L, I, I, P, P, P, L, I, I, I, P],
+    "tie_latent_prep": [I, P, L, I, I, I, I, I, P, P, F, P, P, I, P, P, P, P, I, P],
+    "tie_latent_query_rot": [I, P, L, I, I, P, P, I, P, P, L, I, I, I, P],
     "tie_head_gate_mul": [I, P, L, P, L, I, I, I, P],
-    "tie_attention_latent_prompt": [P, L, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P],
+    "tie_attention_latent_prompt": [P, L, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
     "tie_attention_latent_split": [P, L, P, P, P, P, I, I, I, I, I, I, F, P, I, I, I, P, P],
     "tie_add_concat": [I, P, P, P, L, I, P, P, I, I, P],
     "tie_glu_biased": [I, P, P, P, P, I, I, I, I, P],
@@ -93,12 +93,15 @@ _SIGNATURES = {
     "tie_time_mix_out": [I, P, P, L, P, F, P, I, I, I, P, I, P, L, L, P, P, P, P],
     "tie_two_branch_unit": [I, P, P, L, F, F, P],
     "tie_add_layer_norm": [I, P, *_TERMS, P, P, P, F, P, I, I, P],
+    "tie_add_terms_rmsnorm": [I, P, *_TERMS, P, P, F, P, I, I, P],
     "tie_stream_add": [I, P, *_TERMS, P, P, I, I, P],
     "tie_cap_rows": [P, L, I, I, F, P],
     "tie_short_conv_act": [I, P, L, I, I, I, I, I, P, P, P, P, L, L, P, P, P, I, P, L, P],
     "tie_conv_rope_append": [I, P, L, I, I, I, I, I, P, P, P, L, L, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, P],
     "tie_conv_tail": [I, P, L, I, I, I, I, P, P, L, L, P, P, I, P],
     "tie_selective_scan": [I, P, L, P, L, P, L, I, I, P, P, P, P, P, L, P, P, I, I, I, P, I, P],
+    "tie_rope_split": [I, P, L, I, I, I, I, I, I, I, P, P, I, I, P, F, P, P, P, P],
+    "tie_squared_relu": [I, P, P, L, P],
     "tie_act_split": [I, P, L, I, I, I, I, I, I, I, P, P, P, P],
     "tie_attention_kept_rows": [I, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, P, P],
     "tie_attention_kept_split": [I, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, P, P, I, I, I, P, P],

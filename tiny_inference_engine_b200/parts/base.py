@@ -82,6 +82,12 @@ class PositionEncoding(Part):
         kernel can apply, else None (then `apply` is called on q and k)."""
         return None
 
+    def rotation(self):
+        """(table, whether neighbouring dimensions form the pairs) if the encoding is a rotation, for kernels that take either
+        kind of table (float32 inverse frequencies, or float64 turns a position) and either pairing; else None."""
+        table = self.fused_table()
+        return None if table is None else (table, False)
+
     def score_scale(self) -> float:
         """A factor on the attention scores that the encoding asks for (a rotation stretched to longer
         contexts may come with one); the mixer multiplies its softmax scale by it."""

@@ -1,4 +1,4 @@
-"""Gated feed-forwards. SwiGLU: down(silu(gate(h)) * up(h)), silu(g) = g / (1 + exp(-g))
+"""Feed-forwards, most of them gated. SwiGLU: down(silu(gate(h)) * up(h)), silu(g) = g / (1 + exp(-g))
 (src/model/qwen3.cpp:235-238, src/backend/cpu/cpu_backend.cpp:195-207). Gate and up are
 stacked into one weight so that one product reads h once."""
 from __future__ import annotations
@@ -200,6 +200,40 @@ class TwoBranchMLP(FeedForward):
         return self.down(act, out, lambda n: ctx.ws.flat("ffn.out.partial", n, torch.float32, self._partial_capacity))
 
 
+class SquaredReluMLP(FeedForward):
+    """One hidden layer without a gate: down(max(up(h), 0)^2). On the tensor-core path the activation happens in the epilogue of
+    the first product (in its reduction where k is split), on the float32 accumulator; else a kernel of its own does it. params:
+    `hidden_size`, `intermediate_size`, and the tensors' names (`up`, `down`) after `prefix`."""
+    launches_only = True
+
+    def __init__(self, spec, dtype, prefix: str = ""):
+        p = spec.params
+        self.prefix = prefix + p.get("prefix", "")
+        self.hidden, self.inter = int(p["hidden_size"]), int(p["intermediate_size"])
+        self.names = tuple(self.prefix + p.get(k, k) for k in ("up", "down"))
+        self.dtype = dtype
+        self._partial_capacity = None
+
+    def needs(self):
+        u, d = self.names
+        return {u: TensorNeed((self.inter, self.hidden)), d: TensorNeed((self.hidden, self.inter))}
+
+    def bind(self, get):
+        u, d = self.names
+        self.up = ops.bound_gemm(to_compute(get(u), self.dtype).contiguous(), silu=ops.SQUARED_RELU)
+        self.down = ops.bound_gemm(to_compute(get(d), self.dtype).contiguous())
+        self.w_up, self.w_down = self.up.w, self.down.w
+
+    def forward(self, h, ctx):
+        T = h.shape[0]
+        act = ctx.ws.rows("ffn.act", T, self.inter, self.dtype)
+        self.up(h, act)
+        out = ctx.ws.rows("ffn.out", T, self.hidden, self.dtype)
+        if self._partial_capacity is None:
+            self._partial_capacity = ops.partial_capacity(ctx.ws.max_rows, self.down.N, self.down.K)
+        return self.down(act, out, lambda n: ctx.ws.flat("ffn.out.partial", n, torch.float32, self._partial_capacity))
+
+
 class FeedForwardSum(FeedForward):
     """Feed-forwards side by side on the same input, summed: routed experts beside a shared one that every token passes. The
     sum is handed on as an `ops.ScaledSum`: the residual add that follows forms it in float32. Their outputs must lie in
@@ -226,6 +260,7 @@ class FeedForwardSum(FeedForward):
 
 register_part("feed_forward", "swiglu", SwiGLU, replace=True)
 register_part("feed_forward", "feed_forward_sum", FeedForwardSum, replace=True)
+register_part("feed_forward", "squared_relu_mlp", SquaredReluMLP, replace=True)
 register_part("feed_forward", "two_branch_mlp", TwoBranchMLP, replace=True)
 register_part("feed_forward", "biased_glu", BiasedGLU, replace=True)
 register_part("feed_forward", "clamped_glu", ClampedGLU, replace=True)

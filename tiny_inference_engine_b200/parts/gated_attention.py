@@ -5,10 +5,10 @@
     q, k   = rotation of the first `rotary_dim` dimensions of each head (the position part's table)
     v      = (1 - lambda) v + lambda v_first                              `value_mix` "blend"; "source" keeps v as v_first
     k, v  -> cache pages (keys of `head_dim`, values of `value_dim`)
-    out    = (softmax(scale q k^T over the last `window` keys) v * sigmoid(gate)) Wo^T + bo
+    out    = (softmax(scale q k^T over the last `window` keys) v * sigmoid(gate)) Wo^T + bo      a gate per output channel, or per head
 
 Every size and constant is a parameter, and each option can be left out (`bias`, `span_norm`, `output_gate`,
-`value_mix`, `window` 0 = all keys). The values that a "source" layer computes for the tokens of a step stay in a
+`value_mix`, `window` 0 = all keys); `output_gate` is "channel" (or True), "head", or None. The values that a "source" layer computes for the tokens of a step stay in a
 workspace buffer that "blend" layers of the same step read: they belong to the same tokens, so nothing of it is
 cached. The output product's bias is left to the block (`output_bias`), which adds it in float32.
 """
@@ -24,6 +24,7 @@ from ..weights.loader import TensorNeed
 from .attention import MAX_SPLITS, NUM_SMS, SPLIT_KEYS, decode_splits
 from .base import CacheNeed, Mixer, build_part, register_part, to_compute
 
+_GATES = {None: None, False: None, True: "channel", "channel": "channel", "head": "head"}
 _MIX_MODES = {None: 0, "none": 0, "source": 1, "blend": 2}
 
 
@@ -42,7 +43,9 @@ class GatedWindowAttention(Mixer):
         self.eps = float(p.get("eps", 1e-6))
         self.bias = bool(p.get("bias", False))
         self.span_norm = bool(p.get("span_norm", False))
-        self.output_gate = bool(p.get("output_gate", False))
+        if p.get("output_gate") not in _GATES:
+            raise InvalidArgument(f"output_gate must be channel, head or None, got {p.get('output_gate')!r}")
+        self.output_gate = _GATES[p.get("output_gate")]
         if p.get("value_mix") not in _MIX_MODES:
             raise InvalidArgument(f"value_mix must be one of none, source, blend; got {p.get('value_mix')!r}")
         self.mix_mode = _MIX_MODES[p.get("value_mix")]
@@ -65,7 +68,8 @@ class GatedWindowAttention(Mixer):
         self.k_off = _up8(self.q_dim)
         self.v_off = self.k_off + _up8(self.k_dim)
         self.g_off = self.v_off + _up8(self.v_dim)
-        self.width = self.g_off + (_up8(self.o_dim) if self.output_gate else 0)
+        self.gates = {"channel": self.o_dim, "head": self.heads, None: 0}[self.output_gate]
+        self.width = self.g_off + _up8(self.gates)
         self.output_bias = None
 
     # -- weights
@@ -83,7 +87,7 @@ class GatedWindowAttention(Mixer):
             n.update({self._name("q.norm"): TensorNeed((self.q_dim,), "norm"),
                       self._name("k.norm"): TensorNeed((self.k_dim,), "norm")})
         if self.output_gate:
-            n[self._name("g")] = TensorNeed((self.heads * self.value_dim, D))
+            n[self._name("g")] = TensorNeed((self.heads * (self.value_dim if self.output_gate == "channel" else 1), D))
         # only a blending layer reads the weight; a checkpoint may carry it for the others too (the source layer's
         # is never used), so there it is accepted and ignored
         n[self._name("vmix")] = TensorNeed((), "norm", optional=self.mix_mode != 2)
@@ -95,7 +99,9 @@ class GatedWindowAttention(Mixer):
         for leaf, off, n in (("q", self.q_off, self.q_dim), ("k", self.k_off, self.k_dim), ("v", self.v_off, self.v_dim)):
             stacked[off:off + n] = to_compute(get(self._name(leaf)), self.dtype)
         H, Dv, Do = self.heads, self.value_dim, self.out_dim
-        if self.output_gate:      # head h's gate rows at h * out_dim (rows of the padding stay zero: they gate zeros)
+        if self.output_gate == "head":
+            stacked[self.g_off:self.g_off + H] = to_compute(get(self._name("g")), self.dtype)
+        elif self.output_gate:    # head h's gate rows at h * out_dim (rows of the padding stay zero: they gate zeros)
             stacked[self.g_off:self.g_off + self.o_dim].view(H, Do, self.hidden)[:, :Dv] = \
                 to_compute(get(self._name("g")), self.dtype).view(H, Dv, self.hidden)
         self.gemm_in = ops.bound_gemm(stacked, split_many=False)
@@ -129,20 +135,22 @@ class GatedWindowAttention(Mixer):
             raise InvalidArgument("this attention computes its own keys and values: it cannot read another entry's cache")
         proj = ctx.ws.rows("gattn.proj", T, self.width, self.dtype)
         self.gemm_in(h, proj)
-        table = None if self.position.is_identity else self.position.fused_table()
+        table, neighbours = (None if self.position.is_identity else self.position.rotation()) or (None, False)
         if table is None and not self.position.is_identity:
             raise InvalidArgument("this attention takes a rotation by a frequency table (or none) as its position encoding")
         v_first = ctx.ws.rows("gattn.v_first", T, self.v_dim, torch.float32) if self.mix_mode else None
         ops.qkv_span_prep(proj, self.q_off, self.k_off, self.v_off, self.bq, self.bk, self.bv, self.wq, self.wk, self.eps,
-                          table, ctx.positions, g.slots, cache.k, cache.v, H, G, Dk, Dv, self.mix_mode, v_first, self.lam)
+                          table, ctx.positions, g.slots, cache.k, cache.v, H, G, Dk, Dv, self.mix_mode, v_first, self.lam, neighbours=neighbours)
         attn = ctx.ws.rows("gattn.out", T, self.o_dim, self.dtype)
         q = proj[:, :self.q_dim]
         if Dk == Do and ops.attention_decode_tma_takes(q, H, G, Dk, cache.k.shape[2]):
             self._attend_tensor_cores(q, attn, ctx, g, cache)
         else:
             self._attend_cuda_cores(q, attn, ctx, g, cache)
-        if self.output_gate:
-            ops.sigmoid_gate_mul(attn, proj[:, self.g_off:self.g_off + self.o_dim])
+        if self.output_gate == "channel":
+            ops.sigmoid_gate_mul(attn, proj[:, self.g_off:self.g_off + self.gates])
+        elif self.output_gate == "head":
+            ops.head_gate_mul(attn, proj[:, self.g_off:self.g_off + self.gates], H, Do)
         out = ctx.ws.rows("mixer.out", T, self.hidden, self.dtype)
         if self._capacity is None:
             self._capacity = ops.partial_capacity(ctx.ws.max_rows, self.gemm_o.N, self.gemm_o.K)

@@ -21,7 +21,7 @@ import torch
 from .. import ops
 from ..errors import InvalidArgument
 from ..weights.loader import TensorNeed
-from .base import Mixer, StateNeed, register_part, to_compute
+from .base import Mixer, StateNeed, build_part, register_part, to_compute
 
 
 def _up8(n: int) -> int:
@@ -114,13 +114,16 @@ class GatedLinearAttention(Mixer):
 class ConstantDecayAttention(Mixer):
     """Linear attention whose matrix state decays with one constant per head:
 
-        q, k, v = silu(h Wq^T), silu(h Wk^T), silu(h Wv^T)
+        q, k, v = silu(h Wq^T), silu(h Wk^T), silu(h Wv^T)         or, with `activation` None, as they are, q and k rotated by the
+                                                                   position and k times `k_scale`
         S <- decay_h S + k v^T;   o = S^T q                        the read-out sees the token's own write; no other scale
-        out     = ((o / rms(o) over ALL heads together) * w_norm * sigmoid(h Wg^T)) Wo^T
+        out     = ((o / rms(o)) * w_norm * gate(h Wg^T)) Wo^T      rms over ALL heads together or per head (`norm_per_head`), with
+                                                                   or without a weight (`norm_weight`), gate a sigmoid or a SiLU
 
     S (float32 [dim, value_dim] per head, zero at the start of a sequence) is a request's state. The four projections are one
     stacked product; everything behind them up to the gate is float32. params: `hidden_size`, `num_heads`, `head_dim`,
-    `value_dim`, `decay` (a number per head), `eps`."""
+    `value_dim`, `decay` (a number per head), `eps`; `activation` ("silu" or None), `position` (a part of the position family, or
+    None), `k_scale` (1), `norm_per_head` (False), `norm_weight` (True), `gate` ("sigmoid" or "silu")."""
     launches_only = False
     graph_safe = True
 
@@ -131,6 +134,14 @@ class ConstantDecayAttention(Mixer):
         self.dim, self.vdim = int(p["head_dim"]), int(p["value_dim"])
         self.eps = float(p.get("eps", 1e-6))
         self.decay_values = [float(d) for d in p["decay"]]
+        self.activation, self.k_scale = p.get("activation", "silu"), float(p.get("k_scale", 1.0))
+        self.position = build_part("position", p["position"], dtype, prefix=self.prefix) if p.get("position") else None
+        self.norm_per_head, self.norm_weight = bool(p.get("norm_per_head", False)), bool(p.get("norm_weight", True))
+        if self.activation not in ("silu", None) or p.get("gate", "sigmoid") not in ("sigmoid", "silu"):
+            raise InvalidArgument(f"constant-decay attention: no activation {self.activation!r} or gate {p.get('gate')!r}")
+        self.gate = ops.GATE_SILU if p.get("gate") == "silu" else ops.GATE_SIGMOID
+        if self.activation and (self.position is not None or self.k_scale != 1.0):
+            raise InvalidArgument("constant-decay attention: a rotation or a factor on the keys goes without an activation")
         if min(self.heads, self.vdim) <= 0 or not 0 < self.dim <= 256 or len(self.decay_values) != self.heads:
             raise InvalidArgument(f"constant-decay attention: bad sizes heads={self.heads} dim={self.dim} (1 to 256) vdim={self.vdim} "
                                   f"with {len(self.decay_values)} decays")
@@ -144,8 +155,13 @@ class ConstantDecayAttention(Mixer):
 
     def needs(self):
         D, n = self.hidden, lambda leaf: self.prefix + leaf
-        return {n("q"): TensorNeed((self.nqk, D)), n("k"): TensorNeed((self.nqk, D)), n("v"): TensorNeed((self.nv, D)),
-                n("g"): TensorNeed((self.nv, D)), n("o"): TensorNeed((D, self.nv)), n("norm"): TensorNeed((self.nv,), "norm")}
+        t = {n("q"): TensorNeed((self.nqk, D)), n("k"): TensorNeed((self.nqk, D)), n("v"): TensorNeed((self.nv, D)),
+             n("g"): TensorNeed((self.nv, D)), n("o"): TensorNeed((D, self.nv))}
+        if self.norm_weight:
+            t[n("norm")] = TensorNeed((self.vdim if self.norm_per_head else self.nv,), "norm")
+        if self.position is not None:
+            t.update(self.position.needs())
+        return t
 
     def bind(self, get):
         n = lambda leaf: self.prefix + leaf
@@ -156,8 +172,10 @@ class ConstantDecayAttention(Mixer):
         self.w_in = self.gemm_in.w
         self.gemm_o = ops.bound_gemm(to_compute(get(n("o")), self.dtype).contiguous(), split_many=True)
         self.w_o = self.gemm_o.w
-        self.norm_w = get(n("norm")).to(torch.float32).contiguous()
-        self.decay = torch.tensor([self.decay_values], dtype=torch.float32, device=self.norm_w.device)      # one row for every token
+        self.norm_w = get(n("norm")).to(torch.float32).contiguous() if self.norm_weight else None
+        self.decay = torch.tensor([self.decay_values], dtype=torch.float32, device=stacked.device)      # one row for every token
+        if self.position is not None:
+            self.position.bind(get)
         self._capacity = None
 
     def state_need(self):
@@ -172,13 +190,22 @@ class ConstantDecayAttention(Mixer):
         qn = ctx.ws.rows("cda.q", T, self.nqk, torch.float32)
         kn = ctx.ws.rows("cda.k", T, self.nqk, torch.float32)
         vn = ctx.ws.rows("cda.v", T, self.nv, torch.float32)
-        ops.act_split(proj, self.q_off, self.k_off, self.v_off, qn, kn, vn)
+        if self.activation:
+            ops.act_split(proj, self.q_off, self.k_off, self.v_off, qn, kn, vn)
+        else:
+            table, neighbours = None, False
+            if self.position is not None and not self.position.is_identity:
+                table, neighbours = self.position.rotation() or (None, False)
+                if table is None:
+                    raise InvalidArgument("constant-decay attention takes a rotation by a frequency table (or none) as its position encoding")
+            ops.rope_split(proj, self.q_off, self.k_off, self.v_off, H, dim, table, ctx.positions, self.k_scale, qn, kn, vn, neighbours)
         o = ctx.ws.rows("cda.o", T, self.nv, torch.float32)
         ops.delta_rule(qn, kn, vn, None, self.decay.expand(T, H), state, self.state_floats, proj, self.q_off, self.k_off, self.v_off,
                        ctx.query_start, ctx.state_slots, ctx.S, H, H, dim, vdim, 1, o, plain=True, decay_per_head=True,
                        single=ctx.multi_seqs == 0)
         gated = ctx.ws.rows("cda.gated", T, self.nv, self.dtype)
-        ops.head_norm_gate(o, proj[:, self.g_off:self.g_off + self.nv], self.norm_w, self.eps, gated, 1, self.nv, ops.GATE_SIGMOID)
+        norm_heads, norm_size = (H, vdim) if self.norm_per_head else (1, self.nv)
+        ops.head_norm_gate(o, proj[:, self.g_off:self.g_off + self.nv], self.norm_w, self.eps, gated, norm_heads, norm_size, self.gate)
         out = ctx.ws.rows("mixer.out", T, self.hidden, self.dtype)
         if self._capacity is None:
             self._capacity = ops.partial_capacity(ctx.ws.max_rows, self.gemm_o.N, self.gemm_o.K)

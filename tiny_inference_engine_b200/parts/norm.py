@@ -13,6 +13,7 @@ from .base import Norm, register_part
 class RMSNorm(Norm):
     launches_only = True
     takes_split_sum = True      # add_norm adds the partial sums of a split product itself
+    takes_scaled_sum = True     # and sums of sublayer outputs with factors
     fusable_rms = True          # exactly the formula above, with `weight` (float32) and `eps`
 
     def __init__(self, spec, dtype, prefix: str = ""):
@@ -31,6 +32,8 @@ class RMSNorm(Norm):
     def add_norm(self, x, delta, out, rows=None):
         if isinstance(delta, ops.NormedDelta):      # a sublayer's output that passes a norm of its own on its way in
             ops.add_normed_rmsnorm(x, delta, self.weight, self.eps, out, rows)
+        elif isinstance(delta, ops.ScaledSum):
+            ops.add_terms_rmsnorm(x, delta, self.weight, self.eps, out, rows)
         else:
             ops.add_rmsnorm(x, delta, self.weight, self.eps, out, rows)
 
