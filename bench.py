@@ -262,6 +262,19 @@ def vurazen_config(width, layers, heads, kv_heads, ff, vocab, window=1024, vdim=
             "loop": {"start": layers // 2, "stop": layers, "times": 2}, "norm": {"eps": 1e-6}, "vocab": vocab, "width": width}
 
 
+def sebalorn_config(width, layers, heads, kv_heads, ff, vocab, vdim=128):
+    """Latent attention, grouped-query attention and retention in turn, each over all earlier tokens, at the sizes of a Qwen3
+    layer, every layer with a dense feed-forward; the second half of the layers runs twice."""
+    kinds = [{"type": "latent_attention", "mixer": {"dim": 128, "heads": heads, "kv_rank": 512, "q_rank": 1536, "rot": {"base": 1000000.0, "dims": 64},
+                                                    "rot_dim": 64, "scale": 192 ** -0.5, "vdim": 128}},
+             {"type": "attention", "mixer": {"dim": 128, "heads": heads, "kv_heads": kv_heads, "rot": {"base": 1000000.0, "dims": 64},
+                                             "scale": 128 ** -0.5, "vdim": vdim}},
+             {"type": "retention", "mixer": {"dim": 128, "heads": heads, "rot": {"base": 1000000.0, "dims": 128}, "vdim": vdim,
+                                             "decay": [1.0 - 2.0 ** -(3 + 6 * h / heads) for h in range(heads)]}}]
+    return {"architecture": "Sebalorn", "embedding": {"scale": 12.0}, "layers": [dict(kinds[i % 3], mlp={"ff": ff, "kind": "dense"}) for i in range(layers)],
+            "logit_softcap": 30.0, "loop": {"start": layers // 2, "stop": layers, "times": 2}, "norm": {"eps": 1e-6}, "vocab": vocab, "width": width}
+
+
 DESIGN_SIZES = {     # name: (width, layers, heads, kv heads, feed-forward, vocab)
     "2048x16": (2048, 16, 16, 8, 6144, 151936),
     "4096x8": (4096, 8, 32, 8, 12288, 151936),
@@ -284,13 +297,15 @@ def design_bench(args) -> dict:
         width, layers, heads, kv_heads, ff, vocab = DESIGN_SIZES[size]
         if args.layers:
             layers = args.layers
-        configs = {"misudra": misudra_config(width, layers * 2 // 3, heads, kv_heads, ff, vocab)} if args.design in ("misudra", "lufatar", "vurazen") else {}
+        configs = {"misudra": misudra_config(width, layers * 2 // 3, heads, kv_heads, ff, vocab)} if args.design in ("misudra", "lufatar", "vurazen", "sebalorn") else {}
         if args.design == "subivik":
             configs = {"subivik": subivik_config(width, layers, heads, kv_heads, ff, vocab, vdim=args.design_vdim)}
         if args.design == "lufatar":
             configs = {"lufatar": lufatar_config(width, layers * 2 // 3, heads, kv_heads, ff, vocab, vdim=args.design_vdim), **configs}
         if args.design == "vurazen":
             configs = {"vurazen": vurazen_config(width, layers * 2 // 3, heads, kv_heads, ff, vocab, vdim=args.design_vdim), **configs}
+        if args.design == "sebalorn":
+            configs = {"sebalorn": sebalorn_config(width, layers * 2 // 3, heads, kv_heads, ff, vocab, vdim=args.design_vdim), **configs}
         configs.update({"dugazen": dugazen_config(width, layers, heads, kv_heads, ff, vocab, vdim=args.design_vdim),
                    "qwen3": dict(QWEN3_8B, hidden_size=width, intermediate_size=ff, num_hidden_layers=layers,
                                  num_attention_heads=heads, num_key_value_heads=kv_heads, vocab_size=vocab)})
@@ -367,7 +382,7 @@ def design_bench(args) -> dict:
             torch.cuda.empty_cache()
         rows.append(row)
     return {"design": args.design, "beside": ("misudra, dugazen and qwen3 at equal width, heads and feed-forward and as many layer runs "
-                                              "(two thirds of the layers, the second half run twice)" if args.design in ("lufatar", "vurazen") else
+                                              "(two thirds of the layers, the second half run twice)" if args.design in ("lufatar", "vurazen", "sebalorn") else
                                               "dugazen and qwen3 at equal width, heads and feed-forward and as many layer runs "
                                               "(two thirds of the layers, the second half run twice)" if args.design == "misudra" else
                                               "qwen3 at equal width, layers, heads and feed-forward"), "dtype": "bf16",
@@ -395,11 +410,11 @@ def main() -> int:
     ap.add_argument("--profile", choices=["decode", "prefill", "mixed"], help="run two steps of one kind (mixed: 30 requests "
                     "decoding at context 2,048 beside a 482-token portion of a prompt, the serving default of 512 tokens a step), kernel by kernel, between "
                     "cudaProfilerStart/Stop (for ncu --profile-from-start off) and print no bench line")
-    ap.add_argument("--design", choices=["dugazen", "misudra", "lufatar", "subivik", "vurazen"], help="prefill and decode throughput of that design beside Qwen3 at equal "
+    ap.add_argument("--design", choices=["dugazen", "misudra", "lufatar", "subivik", "vurazen", "sebalorn"], help="prefill and decode throughput of that design beside Qwen3 at equal "
                     "sizes (a line of its own; the default workload and its line stay as they are)")
     ap.add_argument("--design-size", choices=sorted(DESIGN_SIZES), help="--design: one size only")
     ap.add_argument("--design-vdim", type=int, default=128, help="--design: size of a value head (keys have 128)")
-    ap.add_argument("--design-only", choices=["dugazen", "misudra", "lufatar", "subivik", "vurazen", "qwen3"], help="--design: one of the two models only")
+    ap.add_argument("--design-only", choices=["dugazen", "misudra", "lufatar", "subivik", "vurazen", "sebalorn", "qwen3"], help="--design: one of the two models only")
     args = ap.parse_args()
 
     if args.design:

@@ -60,11 +60,19 @@ _act = None       # with `bfloat16_activations()`: rounds what a 16-bit pipeline
 class bfloat16_activations:
     """Within this context the outputs of `linear`, of the norms and of other steps that feed a matrix product are rounded
     to bfloat16 (the weights of the tests are bfloat16 values already): the distance to the exact result is the noise that
-    a pipeline with 16-bit activations cannot avoid, which is what a tolerance for such a pipeline is measured against."""
+    a pipeline with 16-bit activations cannot avoid, which is what a tolerance for such a pipeline is measured against. With
+    `draw`, random relative errors of up to 2^-9 (half a unit of bfloat16) take the place of the rounding."""
+
+    def __init__(self, draw=None):
+        self.draw = draw
 
     def __enter__(self):
         global _act
-        _act = lambda y: round_bf16(y).astype(np.float64)
+        if self.draw is None:
+            _act = lambda y: round_bf16(y).astype(np.float64)
+        else:
+            rng = np.random.default_rng(self.draw)
+            _act = lambda y: f64(y) * (1.0 + rng.uniform(-2.0 ** -9, 2.0 ** -9, np.shape(y)))
 
     def __exit__(self, *exc):
         global _act

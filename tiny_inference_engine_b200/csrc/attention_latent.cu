@@ -97,6 +97,25 @@ __global__ void head_gate_mul_kernel(T* __restrict__ y, long long y_stride, cons
   st(p, ld(p) * (1.0f / (1.0f + expf(-g))));
 }
 
+// Heads of whole 16-byte pieces: one piece a thread.
+template <typename T>
+__global__ void __launch_bounds__(256) head_gate_mul_vec_kernel(T* __restrict__ y, long long y_stride, const T* __restrict__ gate,
+                                                                long long gate_stride, int pieces, int head_size, long long total) {
+  pdl_sync();
+  constexpr int V = Vec16<T>::N;
+  const long long idx = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (idx >= total) return;
+  const long long t = idx / pieces;
+  const int c = static_cast<int>(idx - t * pieces) * V;
+  const float g = 1.0f / (1.0f + expf(-ld(gate + t * gate_stride + c / head_size)));
+  T* p = y + t * y_stride + c;
+  Vec16<T> v;
+  v.load(p);
+#pragma unroll
+  for (int e = 0; e < V; ++e) v.v[e] *= g;
+  v.store(p);
+}
+
 }  // namespace tie
 
 using namespace tie;
@@ -148,6 +167,18 @@ TIE_API int tie_head_gate_mul(int dtype, void* y, long long y_stride, const void
   TIE_REQUIRE(heads > 0 && head_size > 0, "head_gate_mul: bad sizes heads=%d head_size=%d", heads, head_size);
   const long long total = static_cast<long long>(tokens) * heads * head_size;
   if (total <= 0) return kOk;
+  const int vec = dtype == TIE_F32 ? 4 : 8;
+  if (head_size % vec == 0 && y_stride % vec == 0 && reinterpret_cast<uintptr_t>(y) % 16 == 0 && (dtype == TIE_F32 || dtype == TIE_BF16)) {
+    const int pieces = heads * head_size / vec;
+    const long long n = static_cast<long long>(tokens) * pieces;
+    if (dtype == TIE_F32)
+      TIE_LAUNCH((head_gate_mul_vec_kernel<float>), ceil_div(n, 256), 256, 0, s, static_cast<float*>(y), y_stride, static_cast<const float*>(gate),
+                 gate_stride, pieces, head_size, n);
+    else
+      TIE_LAUNCH((head_gate_mul_vec_kernel<__nv_bfloat16>), ceil_div(n, 256), 256, 0, s, static_cast<__nv_bfloat16*>(y), y_stride,
+                 static_cast<const __nv_bfloat16*>(gate), gate_stride, pieces, head_size, n);
+    TIE_RETURN_LAUNCH("head_gate_mul");
+  }
   if (dtype == TIE_F32) {
     TIE_LAUNCH((head_gate_mul_kernel<float>), ceil_div(total, 256), 256, 0, s, static_cast<float*>(y), y_stride,
                static_cast<const float*>(gate), gate_stride, heads * head_size, head_size, total);

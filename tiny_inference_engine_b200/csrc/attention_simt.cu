@@ -440,9 +440,9 @@ static size_t group_split_smem(const AttnArgs& a, int* warps, int* k_pad) {
   return bytes <= 96 * 1024 ? bytes : 0;
 }
 
-// Merge of the splits of one (sequence, head), in split order: one block each. The weights
-// exp(m_i - m) of the splits are computed once into shared memory, then every thread sums its
-// dims over the splits.
+// Merge of the splits of one (sequence, head), in split order: one block for each piece of
+// kMergeThreads dims of it. The weights exp(m_i - m) of the splits are computed once into shared
+// memory, then every thread sums its dim over the splits.
 constexpr int kMergeThreads = 128;
 constexpr int kMergeMaxSplits = 256;
 
@@ -462,7 +462,7 @@ __global__ void __launch_bounds__(kMergeThreads) attention_merge_kernel(AttnArgs
   T* o = static_cast<T*>(a.out) + at;
   float* of = static_cast<float*>(a.out) + at;
   if (pos < 0) {  // a padding sequence: no keys, zeros
-    for (int d = threadIdx.x; d < a.head_dim; d += kMergeThreads) {
+    for (int d = blockIdx.y * kMergeThreads + threadIdx.x; d < a.head_dim; d += gridDim.y * kMergeThreads) {
       if (a.out_f32) of[d] = 0.0f;
       else st(o + d, 0.0f);
     }
@@ -488,13 +488,16 @@ __global__ void __launch_bounds__(kMergeThreads) attention_merge_kernel(AttnArgs
     if (threadIdx.x == 0) inv_l = l > 0.0f ? 1.0f / l : 0.0f;
   }
   __syncthreads();
-  for (int d = threadIdx.x; d < a.head_dim; d += kMergeThreads) {
+  for (int d = blockIdx.y * kMergeThreads + threadIdx.x; d < a.head_dim; d += gridDim.y * kMergeThreads) {
     float acc = 0.0f;
+#pragma unroll 8
     for (int i = 0; i < splits; ++i) acc = fmaf(src[i * stride + d], weight[i], acc);
     if (a.out_f32) of[d] = acc * inv_l;
     else st(o + d, acc * inv_l);
   }
 }
+
+inline dim3 merge_grid(long long items, int dims) { return dim3(static_cast<unsigned>(items), ceil_div(dims, kMergeThreads)); }
 
 template <typename T>
 int launch_attention(const AttnArgs& a, const int* row_seq_unused, const int* seq_list, int n_list, int split_keys,
@@ -523,7 +526,7 @@ int launch_attention(const AttnArgs& a, const int* row_seq_unused, const int* se
         } else                                                                                                   \
         TIE_LAUNCH((attention_split_kernel<T, D>), dim3(ceil_div(items, warps), max_splits), warps * 32, smem, s,           \
             a, seq_list, n_list, split_keys, max_splits, scratch);                                               \
-        TIE_LAUNCH((attention_merge_kernel<T>), static_cast<int>(items), kMergeThreads, 0, s, merge_args, seq_list, n_list, split_keys, \
+        TIE_LAUNCH((attention_merge_kernel<T>), merge_grid(items, merge_args.head_dim), kMergeThreads, 0, s, merge_args, seq_list, n_list, split_keys, \
                                                                                     max_splits, scratch);         \
       }                                                                                                          \
     }                                                                                                            \
@@ -614,9 +617,9 @@ TIE_API int tie_attention_merge(int dtype, void* out, const int* query_start, co
   a.sink = sink;
   const long long items = static_cast<long long>(n_list) * q_heads;
   if (dtype == TIE_F32) {
-    TIE_LAUNCH((attention_merge_kernel<float>), static_cast<int>(items), kMergeThreads, 0, s, a, seq_list, n_list, split_keys, max_splits, scratch);
+    TIE_LAUNCH((attention_merge_kernel<float>), merge_grid(items, head_dim), kMergeThreads, 0, s, a, seq_list, n_list, split_keys, max_splits, scratch);
   } else if (dtype == TIE_BF16) {
-    TIE_LAUNCH((attention_merge_kernel<__nv_bfloat16>), static_cast<int>(items), kMergeThreads, 0, s, a, seq_list, n_list, split_keys, max_splits, scratch);
+    TIE_LAUNCH((attention_merge_kernel<__nv_bfloat16>), merge_grid(items, head_dim), kMergeThreads, 0, s, a, seq_list, n_list, split_keys, max_splits, scratch);
   } else {
     set_error("attention merge: unknown dtype code %d", dtype);
     return kBadArgument;

@@ -24,12 +24,20 @@ import torch
 from .. import ops
 from ..errors import InvalidArgument
 from ..weights.loader import TensorNeed
-from .attention import MAX_SPLITS, SPLIT_KEYS
+from .attention import MAX_SPLITS, NUM_SMS, SPLIT_KEYS
 from .base import CacheNeed, Mixer, build_part, register_part, to_compute
 
 
-LATENT_SPLIT_KEYS = 128     # keys per split of a sequence that brings one token (two key tiles of the tensor-core kernel; shorter
+LATENT_SPLIT_KEYS = 128     # least keys per split of a sequence that brings one token (two key tiles of the tensor-core kernel; shorter
                             # splits cost the merge more than they save the split kernel)
+LATENT_ROWS = 32            # (token, head) rows of a block of that kernel; one block an SM
+
+
+def latent_split_keys(longest: int, sequences: int, heads: int) -> int:
+    """Keys per split: as few splits as give every SM a block (what a split leaves for the merge is `rank` floats a head), in whole
+    tiles of 64 keys, at least LATENT_SPLIT_KEYS."""
+    want = max(1, NUM_SMS // max(1, sequences * math.ceil(heads / LATENT_ROWS)))
+    return max(LATENT_SPLIT_KEYS, -(-math.ceil(longest / want) // 64) * 64)
 
 
 def _up8(n: int) -> int:
@@ -164,7 +172,7 @@ class LatentAttention(Mixer):
                                             ctx.multi_max_queries, H, self.key_dim, self.rank, self.scale, self.window, self.sink)
             if ctx.single_count > 0:
                 longest = ctx.single_max_context if self.window <= 0 else min(ctx.single_max_context, self.window)
-                split_keys = LATENT_SPLIT_KEYS
+                split_keys = latent_split_keys(longest, ctx.single_count, H)
                 while math.ceil(longest / split_keys) > MAX_SPLITS:
                     split_keys *= 2
                 max_splits = max(1, math.ceil(longest / split_keys))
